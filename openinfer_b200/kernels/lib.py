@@ -74,6 +74,10 @@ _SIGNATURES = {
     "oi_dyt_step": [P, P, P, P, P, I, P, P, P, I, P, I, P, I, I, P],
     "oi_rope_norm_store": [P, I, L, I, I, I, I, I, P, I, L, P, P, I, I, I, F, P, P, P, P, L, I, I, P],
     "oi_moe_small": [I, I],
+    "oi_joint_norm_rope_store": [P, I, L, I, I, I, I, I, I, I, P, P, F, P, P, I, I, P, P, P, P, L, I, P],
+    "oi_sigmoid_attention": [P, L, P, L, P, L, I, P, P, L, I, P, I, P, P, I, I, I, I, F, P, P, P],
+    "oi_slice_sum_gate": [P, P, P, P, I, L, P, L, I, I, P],
+    "oi_mingru_scan": [P, I, L, P, L, I, P, P, L, P, P, P, I, I, I, I, P],
     "oi_latent_rope_store": [P, L, I, I, P, L, I, I, I, I, P, I, F, F, I, P, P, I, P, P, I, I, I, I, P],
     "oi_add2_cast": [P, P, P, P, I, L, P],
     "oi_token_gate": [P, L, I, P, P, I, L, I, I, I, I, P],

@@ -811,3 +811,50 @@ def rope_norm_store(qkv: torch.Tensor, nq: int, nkv: int, hd: int, qk_dim: int, 
         0 if bias_tab is None else bias_tab.shape[0], 0 if bias_tab is None else bias_tab.stride(0), _ptr(cos), _ptr(sin),
         0 if cos is None else cos.shape[1], 0 if cos is None else cos.shape[0], 1 if unit_norm else 0, float(eps), positions.data_ptr(),
         _ptr(slots), _ptr(k_cache), _ptr(v_cache), int(page_stride), int(page_size), 1 if write_kv else 0, _stream()), "rope_norm_store")
+
+
+# ---------------------------------------------------------------------------
+# attention with sigmoid weights (csrc/sigmoid_attention.cu) and the recurrence per channel (csrc/gated_scan.cu)
+# ---------------------------------------------------------------------------
+def joint_norm_rope_store(proj: torch.Tensor, nq: int, nkv: int, hd: int, qk_dim: int, k_off: int, v_off: int, *,
+                          q_norm_w: Optional[torch.Tensor], k_norm_w: Optional[torch.Tensor], eps: float,
+                          cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], positions: torch.Tensor, slots: torch.Tensor,
+                          k_cache: torch.Tensor, v_cache: torch.Tensor, page_stride: int, page_size: int) -> None:
+    """Rows [q | ... k at ``k_off`` ... v at ``v_off`` ...] of a fused projection, heads of ``hd`` numbers of which the first
+    ``qk_dim`` count: q, and k, normed over all heads together (float32 weights [heads * hd]; None: not normed), the first 2 *
+    cos.shape[1] numbers of every head turned in neighbouring pairs; q back in place, k and v (as projected; ``v_off`` may
+    equal ``k_off``) to the rows' page slots."""
+    _cuda(proj, q_norm_w, k_norm_w, cos, sin, positions, slots, k_cache, v_cache)
+    _i32(positions, "joint_norm_rope_store positions")
+    _i32(slots, "joint_norm_rope_store slots")
+    if proj.stride(1) != 1 or proj.shape[1] < max(k_off, v_off) + nkv * hd or k_off < nq * hd:
+        raise KernelError(f"joint_norm_rope_store: rows of {proj.shape[1]} numbers, keys at {k_off}, values at {v_off}")
+    for w, heads in ((q_norm_w, nq), (k_norm_w, nkv)):
+        if w is not None and (w.dtype != torch.float32 or w.numel() != heads * hd or not w.is_contiguous()):
+            raise KernelError("joint_norm_rope_store: a norm weight must hold heads * head_dim float32 numbers")
+    if cos is not None and (cos.dtype != torch.float32 or sin is None or sin.shape != cos.shape or not (cos.is_contiguous() and sin.is_contiguous())):
+        raise KernelError("joint_norm_rope_store: cos / sin must be contiguous float32 tables of one shape")
+    if k_cache.dtype != proj.dtype or v_cache.dtype != proj.dtype or positions.numel() != proj.shape[0] or slots.numel() != proj.shape[0]:
+        raise KernelError("joint_norm_rope_store: the cache must have the rows' dtype, and every row a position and a slot")
+    _lib.check(_lib.load().oi_joint_norm_rope_store(
+        proj.data_ptr(), _code(proj, "joint_norm_rope_store"), proj.stride(0), proj.shape[0], nq, nkv, hd, qk_dim, int(k_off), int(v_off),
+        _ptr(q_norm_w), _ptr(k_norm_w), float(eps), _ptr(cos), _ptr(sin), 0 if cos is None else cos.shape[1],
+        0 if cos is None else cos.shape[0], positions.data_ptr(), slots.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
+        int(page_stride), int(page_size), _stream()), "joint_norm_rope_store")
+
+
+def mingru_scan(out: torch.Tensor, zug: torch.Tensor, col_step: int, bias: torch.Tensor, state: torch.Tensor, ctx) -> torch.Tensor:
+    """The rows of a step through the recurrence S <- (1 - z) S + z c(u), request by request: ``zug`` float32 rows with the gate
+    logits, raw candidates and output gate at columns 0, ``col_step`` and 2 ``col_step``; ``bias`` float32 [2, channels] of the
+    first two; ``state`` float32 [slots, channels], read and left behind; out = S * silu(gate)."""
+    _cuda(out, zug, bias, state)
+    C = out.shape[1]
+    if zug.dtype != torch.float32 or zug.stride(1) != 1 or out.stride(1) != 1 or zug.shape[0] != out.shape[0] \
+            or bias.dtype != torch.float32 or tuple(bias.shape) != (2, C) or not bias.is_contiguous() \
+            or state.dtype != torch.float32 or state.shape[-1] != C or not state.is_contiguous():
+        raise KernelError(f"mingru_scan: zug={tuple(zug.shape)} out={tuple(out.shape)} bias={tuple(bias.shape)} state={tuple(state.shape)}")
+    _lib.check(_lib.load().oi_mingru_scan(
+        out.data_ptr(), _code(out, "mingru_scan"), out.stride(0), zug.data_ptr(), zug.stride(0), int(col_step), bias.data_ptr(),
+        state.data_ptr(), state.stride(0), ctx.cu_seqlens.data_ptr(), ctx.token_req.data_ptr(), ctx.state_slots.data_ptr(),
+        out.shape[0], ctx.num_requests, C, 1 if ctx.decode_only else 0, _stream()), "mingru_scan")
+    return out

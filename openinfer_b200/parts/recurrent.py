@@ -1,4 +1,4 @@
-"""Recurrent mixers whose memory is a matrix per head, kept in the cache manager's state slots.
+"""Recurrent mixers whose memory, a matrix per head or a number per channel, is kept in the cache manager's state slots.
 
 "matrix_memory" (the mLSTM cell of xLSTM): per head C [dim, vdim], a normaliser n [dim] and a running maximum m, all zero
 at a request's start. With i = cap tanh(zi / cap) and f = logsigmoid(cap tanh(zf / cap)) (zi, zf: biased projections):
@@ -16,7 +16,11 @@ gated by sigmoid(Wg2 Wg1 x), projected out.
 head S <- decay_h S + k v^T, read-out S^T q with no other scale; the concatenated heads are RMS-normed together with one
 weight, multiplied by sigmoid(Wg x), projected out.
 
-All run as ONE fused input product whose sums stay float32 (gates, decays and everything else that enters the
+"mingru" (a gated recurrence per channel, minGRU): z = sigmoid(Wz x + bz), u = Wx x + bx, S <- (1 - z) S + z c(u) with
+c(u) = u + 1/2 from zero on and sigmoid(u) below, then Wo (S silu(Wg x)); it has its own kernel (csrc/gated_scan.cu), in
+which one block walks a request's rows for a few channels, a run of rows per warp at a time, so its state needs no second copy.
+
+The matrix memories run as ONE fused input product whose sums stay float32 (gates, decays and everything else that enters the
 recurrence never pass through the model's type), the scan kernel over the step's rows (prompt portions and single tokens
 alike, csrc/recurrent.cu), the norm-and-gate kernel, and the output product. The state lives in two copies that take
 turns, like the short filter's.
@@ -32,7 +36,7 @@ from ..kernels import ops
 from ..kernels.linear import linear
 from .base import CacheBinding, Mixer
 from .registry import register_mixer
-from .spec import GatedDeltaSpec, LinearAttentionSpec, MatrixMemorySpec, ParamInfo
+from .spec import GatedDeltaSpec, LinearAttentionSpec, MatrixMemorySpec, MinGruSpec, ParamInfo
 
 
 def _pad8(n: int) -> int:
@@ -247,4 +251,49 @@ class LinearAttention(Mixer):
         y = torch.empty((x.shape[0], H * V), dtype=x.dtype, device=x.device)
         # the norm runs over all heads together: one "head" of H * V numbers
         ops.head_norm_gate(y, o, z[:, self.off["g"]: self.off["g"] + H * V], self.norm_w, 1, H * V, s.eps, weight_per_head=True)
+        return linear(y, self.w_o, out_dtype=out_dtype)
+
+
+@register_mixer("mingru")
+class MinGru(Mixer):
+    graph_safe = True
+    takes_out_dtype = True
+
+    def __init__(self, spec: MinGruSpec) -> None:
+        super().__init__(spec)
+        if spec.channels <= 0:
+            raise ValueError(f"mingru: {spec.channels} channels")
+        # columns of the fused product: gate logits | raw candidates | output gate, each on an 8-column boundary
+        self.step = _pad8(spec.channels)
+        self.w_in: Optional[torch.Tensor] = None
+        self.w_o: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
+
+    def parameters(self) -> Dict[str, ParamInfo]:
+        s = self.spec
+        C, W = s.channels, s.hidden_size
+        std = W ** -0.5
+        return {s.z_name: ParamInfo((C, W), ("normal", std)), s.z_name + s.bias_suffix: ParamInfo((C,), ("normal_around", 1.0, -1.0)),
+                s.x_name: ParamInfo((C, W), ("normal", std)), s.x_name + s.bias_suffix: ParamInfo((C,), ("normal", 0.5)),
+                s.gate_name: ParamInfo((C, W), ("normal", std)), s.out_name: ParamInfo((W, C), ("normal", C ** -0.5))}
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        s = self.spec
+        C = s.channels
+        z = tensors[s.z_name]
+        w = torch.zeros((3 * self.step, z.shape[1]), dtype=z.dtype, device=z.device)
+        for n, name in enumerate((s.z_name, s.x_name, s.gate_name)):
+            w[n * self.step: n * self.step + C] = tensors[name]
+        self.w_in = w
+        self.w_o = tensors[s.out_name].contiguous()
+        self.bias = torch.stack([tensors[s.z_name + s.bias_suffix], tensors[s.x_name + s.bias_suffix]]).to(torch.float32).contiguous()
+
+    def state_needs(self) -> List[StateNeed]:
+        return [StateNeed((self.spec.channels,), "float32")]
+
+    def forward(self, x: torch.Tensor, ctx, binding: CacheBinding, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+        C = self.spec.channels
+        zug = linear(x, self.w_in, out_dtype=torch.float32)
+        y = torch.empty((x.shape[0], C), dtype=x.dtype, device=x.device)
+        ops.mingru_scan(y, zug, self.step, self.bias, ctx.cache.state_tensor(binding.states[0]), ctx)
         return linear(y, self.w_o, out_dtype=out_dtype)

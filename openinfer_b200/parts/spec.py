@@ -308,6 +308,53 @@ class LinearAttentionSpec:
 
 
 @dataclasses.dataclass(frozen=True)
+class SigmoidAttentionSpec:
+    """Attention without a softmax: key j weighs sigmoid(score + bias_head) in query i's sum (every j <= i), and the weights
+    are not normalised over the keys. Optionally the heads' scores are mixed first, score_h <- sum_g T[h, g] score_g."""
+
+    kind: str = "sigmoid_attention"
+    hidden_size: int = 0
+    num_heads: int = 0
+    num_kv_heads: int = 0
+    qk_dim: int = 0                         # per head: size of queries and keys
+    v_dim: int = 0                          # per head: size of values
+    score_scale: float = 1.0
+    position: PositionSpec = PositionSpec(kind="none")     # neighbouring pairs (``interleaved``) only
+    # > 0: q, and k, are normed over ALL their heads together (one root mean square a row, weights ``*_norm_name``
+    # [heads * qk_dim]) before the rotation, with this eps
+    joint_norm_eps: float = 0.0
+    values_from_keys: bool = False          # the values are the keys as projected, before norm and rotation; no v projection
+    mix_heads: bool = False                 # ``mix_name`` [heads, heads]
+    score_bias: bool = False                # ``bias_name`` [heads]
+    output_gate: bool = False               # every output number times sigmoid(W_g x) (``gate_name`` [heads * v_dim, hidden])
+    q_name: str = "q"
+    k_name: str = "k"
+    v_name: str = "v"
+    q_norm_name: str = "q.norm"
+    k_norm_name: str = "k.norm"
+    mix_name: str = "talk"
+    bias_name: str = "pb"
+    gate_name: str = "g"
+    out_name: str = "o"
+
+
+@dataclasses.dataclass(frozen=True)
+class MinGruSpec:
+    """A gated recurrence per channel whose gates read the current token only (minGRU): z = sigmoid(W_z x + b_z), u = W_x x +
+    b_x, S_t = (1 - z) S_(t-1) + z c(u) with c(u) = u + 1/2 for u >= 0 and sigmoid(u) below; the result is W_o (S * silu(W_g
+    x)). S is float32 state per request, zero at its start."""
+
+    kind: str = "mingru"
+    hidden_size: int = 0
+    channels: int = 0
+    z_name: str = "z"
+    x_name: str = "x"
+    gate_name: str = "g"
+    out_name: str = "o"
+    bias_suffix: str = ".b"
+
+
+@dataclasses.dataclass(frozen=True)
 class ParallelMixerSpec:
     """Two mixers side by side that read the same input; the result is left_scale * left + right_scale * right."""
 
