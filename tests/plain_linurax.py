@@ -39,25 +39,27 @@ def talking_scores(q, k, scale: float, talk):
     return torch.einsum("hg,gij->hij", talk, s)
 
 
-def sigmoid_weights(scores, bias):
-    """[H, T, T] scores and a number per head -> weights sigmoid(score + bias) of the keys j <= i, zero elsewhere."""
+def sigmoid_weights(scores, bias, seen=None):
+    """[H, T, T] scores and a number per head -> weights sigmoid(score + bias) of the keys j <= i, zero elsewhere. ``seen``
+    [T, T] takes the place of j <= i (a test asks what a lost key would do)."""
     T = scores.shape[-1]
-    seen = torch.ones((T, T), dtype=torch.bool).tril()
+    seen = torch.ones((T, T), dtype=torch.bool).tril() if seen is None else seen
     return torch.where(seen, torch.sigmoid(scores + bias[:, None, None]), torch.zeros((), dtype=scores.dtype))
 
 
-def attention(h, p: Dict[str, torch.Tensor], pre: str, m: dict, eps: float):
+def attention(h, p: Dict[str, torch.Tensor], pre: str, m: dict, eps: float, seen=None, stored=lambda t: t):
     T = h.shape[0]
     H, G, d = int(m["heads"]), int(m["kv_heads"]), int(m["dim"])
     q, k = h @ p[pre + "q"].T, h @ p[pre + "k"].T
-    v = k.view(T, G, d)                                    # the keys as projected are the values
+    v = stored(k.view(T, G, d))                            # the keys as projected are the values
     q = rms(q, p[pre + "q.norm"], eps).view(T, H, d)       # one root mean square over all heads together
     k = rms(k, p[pre + "k.norm"], eps).view(T, G, d)
     if m.get("rot"):
         pos = torch.arange(T)
         q = turn_neighbours(q, pos, m["rot"]["base"], int(m["rot"]["dims"]))
         k = turn_neighbours(k, pos, m["rot"]["base"], int(m["rot"]["dims"]))
-    w = sigmoid_weights(talking_scores(q, k, float(m["scale"]), p[pre + "talk"]), p[pre + "pb"])
+    q, k = stored(q), stored(k)
+    w = sigmoid_weights(talking_scores(q, k, float(m["scale"]), p[pre + "talk"]), p[pre + "pb"], seen)
     o = torch.einsum("hij,jhd->ihd", w, v.repeat_interleave(H // G, dim=1)).reshape(T, H * d)
     return (o * torch.sigmoid(h @ p[pre + "g"].T)) @ p[pre + "o"].T
 
@@ -84,9 +86,10 @@ def feed_forward(h, p: Dict[str, torch.Tensor], pre: str):
 
 
 def forward(cfg: dict, p: Dict[str, torch.Tensor], tokens: List[int], layers_out: Optional[list] = None, dtype=torch.float64,
-            round_to=None):
+            round_to=None, seen=None):
     """Logits [T, vocab] of one sequence in ``dtype``; ``layers_out`` collects the stream after every layer. ``round_to``:
-    what the sublayers read is rounded to this type on the way (what a 16-bit engine does at least)."""
+    what the sublayers read, and an attention's queries, keys and values, are rounded to this type on the way (what a 16-bit
+    engine does at least)."""
     p = {k: v.to(dtype) for k, v in p.items()}
     eps = float(cfg["norm"]["eps"])
 
@@ -97,7 +100,7 @@ def forward(cfg: dict, p: Dict[str, torch.Tensor], tokens: List[int], layers_out
     for i, layer in enumerate(cfg["layers"]):
         pre = f"l{i}."
         if layer["type"] == "attention":
-            a = attention(read(x), p, pre + "mix.", layer["mixer"], eps)
+            a = attention(read(x), p, pre + "mix.", layer["mixer"], eps, seen, stored=read)
         elif layer["type"] == "mingru":
             a = mingru(read(x), p, pre + "mix.")
         else:
