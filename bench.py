@@ -26,7 +26,9 @@ every kernel's time per step), one JSON line of its own. ``--design pilonex`` do
 rotated key part under one norm with experts picked by a token table, a shared expert and a side input per token),
 ``--design luzitar`` for the Luzitar design (Dynamic Tanh norms on both sides of every sublayer, linear attention with a
 fixed decay per head, attention normed behind its rotation under a window that keeps the first keys, latent attention whose
-cache a later layer reads, experts chosen by corrected sigmoid scores within the best groups).
+cache a later layer reads, experts chosen by corrected sigmoid scores within the best groups),
+``--design linurax`` for the Linurax design (norms on the sublayers' outputs, attention with sigmoid weights whose heads'
+scores are mixed and whose keys are its values, a gated recurrence per channel), beside Qwen3 and Delunex.
 """
 from __future__ import annotations
 
@@ -515,6 +517,22 @@ def luzitar_configs(key, layers=None):
     return luzitar, design_configs(key, layers)[1], bubalix_configs(key, layers)[0]
 
 
+def linurax_configs(key, layers=None):
+    """Linurax at the same widths and depths: every other layer is a gated recurrence of one and a half times the width, every
+    other one attention with sigmoid weights (per head 128 numbers, a quarter as many kv heads, the whole head rotated); every
+    layer has Qwen3's gated feed-forward. Qwen3 as in ``design_configs``; the third configuration returned is Delunex, the
+    engine's other design with norms on its sublayers' outputs."""
+    width, n_layers, heads, _, _, inter = DESIGN_SIZES[key]
+    n_layers = layers or n_layers
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "rot": {"dims": 128, "base": 500000.0}}
+    lay = [{"type": "attention" if i % 2 else "mingru", "mixer": dict(att) if i % 2 else {"width": 3 * width // 2},
+            "mlp": {"kind": "dense", "ff": inter}} for i in range(n_layers)]
+    linurax = {"architecture": "Linurax", "vocab": DESIGN_VOCAB, "width": width, "embedding": {"scale": 8.0}, "norm": {"eps": 1e-6},
+               "layers": lay}
+    delunex, qwen = design_configs(key, layers)
+    return linurax, qwen, delunex
+
+
 def _part_tensors(torch, part, seen=None):
     """Every tensor a part holds, the tensors of parts inside it included."""
     seen = set() if seen is None else seen
@@ -693,8 +711,10 @@ def design_mode(args, torch, mods, peaks, peaks_src):
             if key not in DESIGN_SIZES:
                 raise SystemExit(f"--design-sizes: unknown size {key!r} (known: {', '.join(DESIGN_SIZES)})")
             rec = {"width": DESIGN_SIZES[key][0], "layers": args.layers or DESIGN_SIZES[key][1]}
-            configs = {"pilonex": pilonex_configs, "bubalix": bubalix_configs, "luzitar": luzitar_configs}.get(args.design, design_configs)(key, args.layers)
-            for arch, cfg in zip((args.design, "qwen3", "bubalix"), configs):      # (a third entry only where the design names one)
+            configs = {"pilonex": pilonex_configs, "bubalix": bubalix_configs, "luzitar": luzitar_configs,
+                       "linurax": linurax_configs}.get(args.design, design_configs)(key, args.layers)
+            third = {"luzitar": "bubalix", "linurax": "delunex"}.get(args.design)      # the engine's closest design, where one is measured too
+            for arch, cfg in zip((args.design, "qwen3", third), configs):
                 b = DesignBench(torch, mods, cfg, args.dtype, CONTEXT, 64, steps + warm + 16)
                 r = {"weights_gb": round(b.runner.model.weight_bytes() / 1e9, 3)}
                 for batch in (1, 8, 64):
@@ -754,7 +774,7 @@ def main() -> int:
     ap.add_argument("--profile", choices=["decode", "prefill", "mixed", "sampler"], default=None,
                     help="run warm-up, then ONE step between cudaProfilerStart/Stop and exit "
                          "(for `ncu --profile-from-start off`); prints no benchmark line")
-    ap.add_argument("--design", default=None, choices=["delunex", "pilonex", "bubalix", "luzitar"],
+    ap.add_argument("--design", default=None, choices=["delunex", "pilonex", "bubalix", "luzitar", "linurax"],
                     help="instead of the headline workload: this design at layer sizes of real models beside Qwen3 at equal "
                          "sizes (decode at batch 1/8/64, a 2,048-token prefill), one JSON line")
     ap.add_argument("--design-sizes", default=None, help="sizes for --design, comma separated (1k, 2k, 4k; default 1k,2k)")

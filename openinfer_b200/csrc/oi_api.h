@@ -161,6 +161,31 @@ OI_API int oi_rope_norm_store(void* qkv, int dtype, long long row_stride, int to
        int max_pos, int unit_norm, float eps, const int* positions, const int* slots, void* k_cache, void* v_cache,
        long long page_stride, int page_size, int write_kv, void* stream);
 
+// sigmoid_attention.cu, sigmoid_attention_mma.cu: attention whose weights are sigmoids, not normalised over the keys, with the
+// heads' scores mixed first: the norm over all heads + rotation of neighbours + cache write in front of it, the general
+// kernel, the tensor-core kernels (bfloat16; work items planned by the caller) and the sum of a row's key slices with the gate
+OI_API int oi_joint_norm_rope_store(void* proj, int dtype, long long row_stride, int tokens, int nq, int nkv, int hd, int qk_dim,
+       int k_off, int v_off, const float* q_w, const float* k_w, float eps, const float* cos_tab, const float* sin_tab, int
+       rot_half, int max_pos, const int* positions, const int* slots, void* k_cache, void* v_cache, long long page_stride, int
+       page_size, void* stream);
+OI_API int oi_sigmoid_attention(const void* q, long long q_stride, void* out, long long out_stride, const void* gate, long long
+       gate_stride, int dtype, const void* k_cache, const void* v_cache, long long page_stride, int page_size, const int*
+       block_table, int bt_stride, const int* token_req, const int* positions, int tokens, int nq, int nkv, int hd, float scale,
+       const float* mix, const float* bias, void* stream);
+OI_API int oi_sigmoid_attention_tile_tokens(int nq, int nkv, int hd);
+OI_API int oi_sigmoid_attention_mma(const void* q, long long q_stride, void* out, long long out_stride, const void* gate, long
+       long gate_stride, const void* k_cache, const void* v_cache, long long page_stride, int page_size, const int* block_table,
+       int bt_stride, const int* cu_seqlens, const int* kv_lens, const int* tile_items, int n_tiles, const int* decode_items,
+       int n_decode, const int* row_base, float* part, int nq, int nkv, int hd, float scale, const float* mix, const float*
+       bias, void* stream);
+OI_API int oi_slice_sum_gate(const float* part, const int* row_splits, const int* row_base, void* out, int dtype, long long
+       out_stride, const void* gate, long long gate_stride, int tokens, int cols, void* stream);
+
+// gated_scan.cu: a gated recurrence per channel, S <- (1 - z) S + z c(u)
+OI_API int oi_mingru_scan(void* out, int out_dtype, long long out_stride, const float* zug, long long stride, int col_step, const
+       float* bias, float* state, long long state_stride, const int* cu_seqlens, const int* token_req, const int* state_slots,
+       int tokens, int requests, int channels, int singles, int longer, void* stream);
+
 // hyper.cu: several residual streams
 OI_API int oi_hyper_step(float* X, int rows, int S, int W, const float* y, const float* y2, float c1, float c2, const
        void* mix, const void* b_out, const void* a_in, int p_dtype, const void* norm_w, int nw_dtype, float eps, float

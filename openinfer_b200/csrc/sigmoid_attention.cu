@@ -60,18 +60,45 @@ __device__ __forceinline__ void norm_and_turn(float (&x)[8], float inv, const fl
 #pragma unroll
     for (int e = 0; e < 8; ++e) x[e] = x[e] * inv * wv[e];
   }
+  const int n0 = d >> 1;
+  if (n0 >= rot_half) return;
+  float c[4], s[4];
+  if (rot_half % 4 == 0) {                     // the angles of four pairs at a time
+    const float4 c4 = *reinterpret_cast<const float4*>(cos_row + n0), s4 = *reinterpret_cast<const float4*>(sin_row + n0);
+    c[0] = c4.x, c[1] = c4.y, c[2] = c4.z, c[3] = c4.w;
+    s[0] = s4.x, s[1] = s4.y, s[2] = s4.z, s[3] = s4.w;
+  } else {
 #pragma unroll
-  for (int e = 0; e < 8; e += 2) {
-    const int n = (d + e) >> 1;
-    if (n >= rot_half) continue;
-    const float c = cos_row[n], s = sin_row[n];
-    const float u = x[e], v = x[e + 1];
-    x[e] = u * c - v * s;
-    x[e + 1] = v * c + u * s;
+    for (int e = 0; e < 4; ++e) {
+      const bool in = n0 + e < rot_half;
+      c[e] = in ? cos_row[n0 + e] : 1.f;
+      s[e] = in ? sin_row[n0 + e] : 0.f;
+    }
+  }
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    const float u = x[2 * e], v = x[2 * e + 1];
+    x[2 * e] = u * c[e] - v * s[e];
+    x[2 * e + 1] = v * c[e] + u * s[e];
   }
 }
 
-template <typename T>
+// Two sums over the block at once. `red` holds 64 floats.
+__device__ __forceinline__ void block_sum2(float& a, float& b, float* red) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = (blockDim.x + 31) >> 5;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    a += __shfl_xor_sync(0xffffffffu, a, o);
+    b += __shfl_xor_sync(0xffffffffu, b, o);
+  }
+  if (lane == 0) red[warp] = a, red[32 + warp] = b;
+  __syncthreads();
+  a = b = 0.f;
+  for (int w = 0; w < warps; ++w) a += red[w], b += red[32 + w];
+}
+
+// kKeep: eights of q | k a thread keeps in registers between the sum and the turn (0: they are read again)
+template <typename T, int kKeep>
 __global__ void __launch_bounds__(kThreads)
 joint_norm_rope_store_kernel(T* __restrict__ proj, long long row_stride, int nq, int nkv, int hd, int qk_dim, int k_off, int v_off,
                              const float* __restrict__ q_w, const float* __restrict__ k_w, float eps,
@@ -79,50 +106,79 @@ joint_norm_rope_store_kernel(T* __restrict__ proj, long long row_stride, int nq,
                              const int* __restrict__ positions, const int* __restrict__ slots, T* __restrict__ k_cache,
                              T* __restrict__ v_cache, long long page_stride, int page_size) {
   pdl_start();
-  __shared__ float red[32];
-  const int t = blockIdx.x;
+  __shared__ float red[64];
+  const int t = blockIdx.x, step = blockDim.x;
   T* row = proj + (size_t)t * row_stride;
   const int q8 = nq * hd / 8, k8 = nkv * hd / 8;
+  const int slot = slots[t];
+  int pos = positions[t];
+  float keep[kKeep ? kKeep : 1][8];
+  auto source = [&](int i) { return i < q8 ? row + (size_t)i * 8 : row + k_off + (size_t)(i - q8) * 8; };
   float q_inv = 1.f, k_inv = 1.f;
-  if (q_w) {
+  if (q_w || kKeep) {
     float qs = 0.f, ks = 0.f;
-    for (int i = threadIdx.x; i < q8 + k8; i += blockDim.x) {
-      float x[8], s = 0.f;
-      load8<T>(i < q8 ? row + (size_t)i * 8 : row + k_off + (size_t)(i - q8) * 8, x);
+    auto add = [&](int i, const float (&x)[8]) {
+      float s = 0.f;
 #pragma unroll
       for (int e = 0; e < 8; ++e) s += x[e] * x[e];
       if (i < q8) qs += s; else ks += s;
+    };
+    if (kKeep) {
+#pragma unroll
+      for (int n = 0; n < kKeep; ++n) {
+        const int i = threadIdx.x + n * step;
+        if (i < q8 + k8) load8<T>(source(i), keep[n]);
+      }
+#pragma unroll
+      for (int n = 0; n < kKeep; ++n)
+        if ((int)threadIdx.x + n * step < q8 + k8) add(threadIdx.x + n * step, keep[n]);
+    } else {
+      for (int i = threadIdx.x; i < q8 + k8; i += step) {
+        float x[8];
+        load8<T>(source(i), x);
+        add(i, x);
+      }
     }
-    qs = block_sum(qs, red);
-    ks = block_sum(ks, red);
-    q_inv = 1.f / sqrtf(qs / (float)(nq * qk_dim) + eps);
-    k_inv = 1.f / sqrtf(ks / (float)(nkv * qk_dim) + eps);
+    if (q_w) {
+      block_sum2(qs, ks, red);
+      q_inv = 1.f / sqrtf(qs / (float)(nq * qk_dim) + eps);
+      k_inv = 1.f / sqrtf(ks / (float)(nkv * qk_dim) + eps);
+    }
   }
-  int pos = positions[t];
   pos = pos < 0 ? 0 : (rot_half > 0 && pos >= max_pos ? max_pos - 1 : pos);      // admission bounds positions
   const float* cr = rot_half > 0 ? cos_tab + (size_t)pos * rot_half : nullptr;
   const float* sr = rot_half > 0 ? sin_tab + (size_t)pos * rot_half : nullptr;
-  const int slot = slots[t];
   const size_t at = slot >= 0 ? (size_t)(slot / page_size) * page_stride + (size_t)(slot % page_size) * nkv * hd : 0;
-  const int total = q8 + (slot >= 0 ? 2 * k8 : 0);              // a padding row stores nothing
-  for (int i = threadIdx.x; i < total; i += blockDim.x) {
-    float x[8];
+  auto finish = [&](int i, float (&x)[8]) {
     if (i < q8) {
       const int c = i * 8;
-      load8<T>(row + c, x);
       norm_and_turn(x, q_inv, q_w ? q_w + c : nullptr, c % hd, cr, sr, rot_half);
       store8(row + c, x);
-    } else if (i < q8 + k8) {
-      const int c = (i - q8) * 8;
-      load8<T>(row + k_off + c, x);
-      norm_and_turn(x, k_inv, k_w ? k_w + c : nullptr, c % hd, cr, sr, rot_half);
-      store8(k_cache + at + c, x);
-    } else {
-      const int c = (i - q8 - k8) * 8;
-      load8<T>(row + v_off + c, x);
-      store8(v_cache + at + c, x);
+      return;
+    }
+    if (slot < 0) return;                                       // a padding row stores nothing
+    const int c = (i - q8) * 8;
+    if (v_off == k_off) store8(v_cache + at + c, x);            // the value is the key as projected
+    norm_and_turn(x, k_inv, k_w ? k_w + c : nullptr, c % hd, cr, sr, rot_half);
+    store8(k_cache + at + c, x);
+  };
+  if (kKeep) {
+#pragma unroll
+    for (int n = 0; n < kKeep; ++n)
+      if ((int)threadIdx.x + n * step < q8 + k8) finish(threadIdx.x + n * step, keep[n]);
+  } else {
+    for (int i = threadIdx.x; i < q8 + k8; i += step) {
+      float x[8];
+      load8<T>(source(i), x);
+      finish(i, x);
     }
   }
+  if (v_off != k_off && slot >= 0)
+    for (int i = threadIdx.x; i < k8; i += step) {
+      float x[8];
+      load8<T>(row + v_off + (size_t)i * 8, x);
+      store8(v_cache + at + (size_t)i * 8, x);
+    }
 }
 
 constexpr int kChunk = 32;     // keys at a time
@@ -194,23 +250,38 @@ sigmoid_attention_kernel(const T* __restrict__ q, long long q_stride, T* __restr
   }
 }
 
-// out[t] = sigmoid(gate[t]) * sum_s part[row_base[t] + s], for the rows whose keys were cut into more than one slice
-template <typename T>
+// out[t] = sigmoid(gate[t]) * sum_s part[row_base[t] + s], for the rows whose keys were cut into more than one slice. kWays
+// neighbouring warps share 128 columns, each adding up every kWays-th slice.
+template <typename T, int kWays>
 __global__ void __launch_bounds__(kThreads)
 slice_sum_gate_kernel(const float* __restrict__ part, const int* __restrict__ row_splits, const int* __restrict__ row_base,
                       T* __restrict__ out, long long out_stride, const T* __restrict__ gate, long long gate_stride, int cols) {
   pdl_start();
+  __shared__ float4 sums[kWays > 1 ? kThreads : 1];
   const int t = blockIdx.x, n = row_splits[t];
   if (n <= 1) return;
+  const int lane = threadIdx.x & 31, way = (threadIdx.x >> 5) % kWays;
+  const int c = ((blockIdx.y * (blockDim.x / (32 * kWays)) + (threadIdx.x >> 5) / kWays) * 32 + lane) * 4;
   const float* p = part + (size_t)row_base[t] * cols;
-  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
-  if (c >= cols) return;
   float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 8
-  for (int s = 0; s < n; ++s) {
-    const float4 v = *reinterpret_cast<const float4*>(p + (size_t)s * cols + c);
-    a.x += v.x, a.y += v.y, a.z += v.z, a.w += v.w;
+  if (c < cols) {
+#pragma unroll 4
+    for (int s = way; s < n; s += kWays) {
+      const float4 v = *reinterpret_cast<const float4*>(p + (size_t)s * cols + c);
+      a.x += v.x, a.y += v.y, a.z += v.z, a.w += v.w;
+    }
   }
+  if (kWays > 1) {
+    sums[threadIdx.x] = a;
+    __syncthreads();
+    if (way != 0) return;
+#pragma unroll
+    for (int w = 1; w < kWays; ++w) {
+      const float4 v = sums[threadIdx.x + w * 32];
+      a.x += v.x, a.y += v.y, a.z += v.z, a.w += v.w;
+    }
+  }
+  if (c >= cols) return;
   float o[4] = {a.x, a.y, a.z, a.w};
 #pragma unroll
   for (int e = 0; e < 4; ++e) {
@@ -234,18 +305,24 @@ OI_API int oi_joint_norm_rope_store(void* proj, int dtype, long long row_stride,
              "joint_norm_rope_store: %d rotated pairs in a head of %d numbers, or no tables", rot_half, hd);
   OI_REQUIRE(positions && slots && k_cache && v_cache && page_size > 0, "joint_norm_rope_store: positions, slots and pages are needed");
   OI_REQUIRE(row_stride % 8 == 0 && page_stride % 8 == 0 && aligned16(proj) && aligned16(k_cache) && aligned16(v_cache) &&
-             aligned16(q_w) && aligned16(k_w), "joint_norm_rope_store: rows and pages must be readable 16 bytes at a time");
+             aligned16(q_w) && aligned16(k_w) && aligned16(cos_tab) && aligned16(sin_tab), "joint_norm_rope_store: rows and pages must be readable 16 bytes at a time");
   if (tokens == 0) return OI_OK;
   cudaStream_t s = (cudaStream_t)stream;
-  const int work = (nq + 2 * nkv) * hd / 8;
-  const int threads = work >= kThreads ? kThreads : ((work + 31) / 32) * 32;
+  // a row's eights over the threads as evenly as whole warps allow, one or two a thread where that suffices
+  const int work = (nq + nkv) * hd / 8, keep = work <= kThreads ? 1 : (work <= 2 * kThreads ? 2 : (work <= 4 * kThreads ? 4 : 0));
+  const int threads = keep ? ((work + keep - 1) / keep + 31) / 32 * 32 : kThreads;
 #define OI_JNRS(T)                                                                                                         \
-  oi_launch(joint_norm_rope_store_kernel<T>, tokens, threads, 0, s, (T*)proj, row_stride, nq, nkv, hd, qk_dim, k_off, v_off, q_w, \
+  do {                                                                                                                     \
+    if (keep == 1) OI_JNRS_K(T, 1); else if (keep == 2) OI_JNRS_K(T, 2); else if (keep == 4) OI_JNRS_K(T, 4); else OI_JNRS_K(T, 0); \
+  } while (0)
+#define OI_JNRS_K(T, KEEP)                                                                                                 \
+  oi_launch(joint_norm_rope_store_kernel<T, KEEP>, tokens, threads, 0, s, (T*)proj, row_stride, nq, nkv, hd, qk_dim, k_off, v_off, q_w, \
             k_w, eps, cos_tab, sin_tab, rot_half, max_pos, positions, slots, (T*)k_cache, (T*)v_cache, page_stride, page_size)
   if (dtype == OI_F32) OI_JNRS(float);
   else if (dtype == OI_BF16) OI_JNRS(bf16);
   else OI_REQUIRE(false, "joint_norm_rope_store: unknown dtype code %d", dtype);
 #undef OI_JNRS
+#undef OI_JNRS_K
   OI_CHECK_LAUNCH();
   return OI_OK;
 }
@@ -282,17 +359,23 @@ OI_API int oi_slice_sum_gate(const float* part, const int* row_splits, const int
                              const void* gate, long long gate_stride, int tokens, int cols, void* stream) {
   OI_REQUIRE(tokens >= 0 && cols > 0 && cols % 4 == 0 && aligned16(part) && row_splits && row_base, "slice_sum_gate: bad arguments");
   if (tokens == 0) return OI_OK;
-  const dim3 grid(tokens, (cols / 4 + kThreads - 1) / kThreads);
-  const int threads = cols / 4 >= kThreads ? kThreads : ((cols / 4 + 31) / 32) * 32;
+  // few rows (of many slices, in a step of single tokens): several warps a column; many rows: one
+  const int ways = tokens <= 256 ? 8 : 1, per_block = kThreads / 32 / ways * 128;
+  const dim3 grid(tokens, (cols + per_block - 1) / per_block);
   cudaStream_t s = (cudaStream_t)stream;
-  if (dtype == OI_F32)
-    oi_launch(slice_sum_gate_kernel<float>, grid, threads, 0, s, part, row_splits, row_base, (float*)out, out_stride,
-              (const float*)gate, gate_stride, cols);
-  else if (dtype == OI_BF16)
-    oi_launch(slice_sum_gate_kernel<bf16>, grid, threads, 0, s, part, row_splits, row_base, (bf16*)out, out_stride, (const bf16*)gate,
-              gate_stride, cols);
-  else
-    OI_REQUIRE(false, "slice_sum_gate: unknown dtype code %d", dtype);
+#define OI_SSG(T)                                                                                                            \
+  do {                                                                                                                       \
+    if (ways == 8)                                                                                                           \
+      oi_launch(slice_sum_gate_kernel<T, 8>, grid, kThreads, 0, s, part, row_splits, row_base, (T*)out, out_stride, (const T*)gate, \
+                gate_stride, cols);                                                                                          \
+    else                                                                                                                     \
+      oi_launch(slice_sum_gate_kernel<T, 1>, grid, kThreads, 0, s, part, row_splits, row_base, (T*)out, out_stride, (const T*)gate, \
+                gate_stride, cols);                                                                                          \
+  } while (0)
+  if (dtype == OI_F32) OI_SSG(float);
+  else if (dtype == OI_BF16) OI_SSG(bf16);
+  else OI_REQUIRE(false, "slice_sum_gate: unknown dtype code %d", dtype);
+#undef OI_SSG
   OI_CHECK_LAUNCH();
   return OI_OK;
 }

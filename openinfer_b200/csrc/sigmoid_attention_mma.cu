@@ -171,9 +171,11 @@ __device__ __forceinline__ float sigmoid_gate(float g) { return __fdividef(1.f, 
 
 // ---------------------------------------------------------------------------------------------
 // Prompt tiles. NQ: quads of heads. NQ warps share four neighbouring tokens: a warp owns one quad of heads, its columns are
-// two tiles of 4 heads x 2 tokens, so a fragment of K or V read from shared memory feeds two products. It hands its raw scores
-// to the other warps through shared memory (lane to lane: the fragments lie alike in all of them) and forms the weights and
-// sums of its own heads. A step is KT x 16 keys. ALIGNED: a quad's query heads share one kv head.
+// two tiles of 4 heads x 2 tokens, so a fragment of K or V read from shared memory feeds two products. A step is KT x 16 keys.
+// The mix needs all heads of a (16 keys, two tokens) at once, so it is shared out the other way round: the warps leave their
+// raw scores in shared memory (lane to lane: the fragments lie alike in all of them), each takes KT of the KT * NQ (16 keys,
+// two tokens, eight output heads), forms their weights and leaves them for the warps that own the heads.
+// ALIGNED: a quad's query heads share one kv head.
 // ---------------------------------------------------------------------------------------------
 constexpr int kTileWarps = 16;
 
@@ -188,7 +190,9 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) sigmoid_tile_kernel(const 
   bf16* const q_sm = q_all + (size_t)warp * 16 * HD;               // this warp's columns: row 8 pair + 2 head + token
   float4* const mail_all = reinterpret_cast<float4*>(q_all + (size_t)kTileWarps * 16 * HD);
   float4* const mail = mail_all + (size_t)group4 * KT * 2 * NQ * 32 + lane;          // [key tile][pair][quad][32 lanes]
-  bf16* const ring = reinterpret_cast<bf16*>(mail_all + (size_t)kTileWarps * KT * 2 * 32);
+  uint2* const wmail_all = reinterpret_cast<uint2*>(mail_all + (size_t)kTileWarps * KT * 2 * 32);
+  uint2* const wmail = wmail_all + (size_t)group4 * KT * 2 * NQ * 32 + lane;         // the weights, in the same order
+  bf16* const ring = reinterpret_cast<bf16*>(wmail_all + (size_t)kTileWarps * KT * 2 * 32);
   const int4 item = p.items[blockIdx.x];
   const int req = item.x, tok0 = item.y, slice = item.z, slices = item.w;
   const int q_start = p.cu_seqlens[req], q_len = p.cu_seqlens[req + 1] - q_start;
@@ -206,18 +210,21 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) sigmoid_tile_kernel(const 
   const int my_row = threadIdx.x / per_row, my_chunk = threadIdx.x % per_row, row_chunks = row_elems / 8;
   const unsigned my_dst = smem_u32(ring) + 2 * swz<HD>(my_row, row_elems, (my_chunk / head_chunks) * HD, my_chunk % head_chunks);
   int requested = 0, rq_slot = 0, rq_key = t_begin * kStep + my_row;
-  auto page_of = [&](int key) { return key < key_end ? bt[key / p.page_size] : 0; };
-  int page = units > 0 ? page_of(rq_key) : 0;
+  // the element where this thread's chunks of a step begin, in K's pages as in V's; the page of the step behind it is looked up
+  // two stages before its use
+  int next_page = units > 0 && rq_key < key_end ? bt[rq_key / p.page_size] : 0;
+  size_t at = 0;
   auto request = [&]() {
     if (requested < units) {
       const bool is_v = requested & 1, valid = rq_key < key_end;
-      const bf16* src = (is_v ? p.v_cache : p.k_cache) + (size_t)page * p.page_stride + (size_t)(rq_key % p.page_size) * row_elems + my_chunk * 8;
+      if (!is_v) {
+        at = (size_t)next_page * p.page_stride + (size_t)(rq_key % p.page_size) * row_elems + my_chunk * 8;
+        next_page = rq_key + kStep < key_end ? bt[(rq_key + kStep) / p.page_size] : 0;
+      }
+      const bf16* src = (is_v ? p.v_cache : p.k_cache) + at;
       const unsigned dst = my_dst + (unsigned)(rq_slot * unit * 2);
       for (int i = 0; i * per_row + my_chunk < row_chunks; ++i) cp_async16_or_zero(dst + i * per_row * 16, src + i * per_row * 8, valid);
-      if (is_v) {
-        rq_key += kStep;
-        if (requested + 1 < units) page = page_of(rq_key);      // used two stages later
-      }
+      if (is_v) rq_key += kStep;
     }
     ++requested;
     rq_slot = rq_slot + 1 == stages ? 0 : rq_slot + 1;
@@ -236,18 +243,29 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) sigmoid_tile_kernel(const 
     if (h < p.nq && tok < tile_toks) v = *reinterpret_cast<const uint4*>(p.q + (size_t)(q_start + tok0 + tok) * p.q_stride + (size_t)h * HD + ch * 8);
     *reinterpret_cast<uint4*>(q_sm + swz<HD>(r, HD, 0, ch)) = v;
   }
-  // The mix's right operand: step s of the sum takes heads 8 s + k in order; of the eight output columns the even ones are
-  // this warp's heads (column 2 t: head t of the quad), the odd ones stay empty.
-  unsigned T0[NQ / 2], T1[NQ / 2];
+  // This warp's share of the mix: item i is output tile it % (NQ / 2) (heads 8 tile ...) of combination it / (NQ / 2) (16 keys
+  // and two tokens: key tile * 2 + pair), it = KT quad + i. The right operand: step s of the sum takes heads 8 s + k in
+  // order; output column n stands for head 8 tile + 4 (n & 1) + (n >> 1), so that a thread's two columns are head t of the
+  // tile's first quad and head t of its second.
+  constexpr int kTiles = NQ / 2;
+  unsigned T0[KT][kTiles], T1[KT][kTiles];
+  float nb[KT][2];
 #pragma unroll
-  for (int s = 0; s < NQ / 2; ++s) {
-    const int n = lane >> 2, h = 4 * quad + (n >> 1), g = 8 * s + (lane & 3);
-    const bool on = (n & 1) == 0 && h < p.nq;
-    T0[s] = __float_as_uint(on && g < p.nq ? p.mix[h * p.nq + g] : 0.f);
-    T1[s] = __float_as_uint(on && g + 4 < p.nq ? p.mix[h * p.nq + g + 4] : 0.f);
+  for (int i = 0; i < KT; ++i) {
+    const int tile = (KT * quad + i) % kTiles, n = lane >> 2, h = 8 * tile + 4 * (n & 1) + (n >> 1);
+#pragma unroll
+    for (int s = 0; s < kTiles; ++s) {
+      const int g = 8 * s + (lane & 3);
+      T0[i][s] = __float_as_uint(h < p.nq && g < p.nq ? p.mix[h * p.nq + g] : 0.f);
+      T1[i][s] = __float_as_uint(h < p.nq && g + 4 < p.nq ? p.mix[h * p.nq + g + 4] : 0.f);
+    }
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int hh = 8 * tile + 4 * u + (lane & 3);
+      nb[i][u] = hh < p.nq ? -p.bias[hh] * kLog2eF : 0.f;
+    }
   }
   const int my_head = 4 * quad + (lane & 3);
-  const float nb = my_head < p.nq ? -p.bias[my_head] * kLog2eF : 0.f;
   const int first_pos = pos0 + 4 * group4, toks = min(4, tile_toks - 4 * group4), last_pos = toks > 0 ? first_pos + toks - 1 : -1;
   float O[2][HD / 16][4];
 #pragma unroll
@@ -274,7 +292,6 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) sigmoid_tile_kernel(const 
   const unsigned ring_at = smem_u32(ring);
   const int tile_bytes = kTile * row_elems * 2;
 
-  unsigned w0[KT][2], w1[KT][2];
   int slot = 0;
   for (int u = 0; u < units; u += 2) {
     const int key0 = (t_begin + (u >> 1)) * kStep;
@@ -321,55 +338,76 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) sigmoid_tile_kernel(const 
               for (int i = 0; i < 2; ++i) mma_bf16(S[kt][i], a[kt][x], b[i][2 * x], b[i][2 * x + 1]);
         }
       }
-      // (everyone has read the last step's mail: two barriers of the block lie between)
+      // (everyone has read the last step's scores: two barriers of the block lie between; the weights likewise)
 #pragma unroll
       for (int kt = 0; kt < KT; ++kt)
 #pragma unroll
         for (int i = 0; i < 2; ++i) mail[((kt * 2 + i) * NQ + quad) * 32] = make_float4(S[kt][i][0], S[kt][i][1], S[kt][i][2], S[kt][i][3]);
       asm volatile("bar.sync %0, %1;\n" ::"r"(group4 + 1), "n"(NQ * 32) : "memory");
       const bool full = key0 + kStep - 1 <= first_pos && toks == 4;
+      constexpr int kShare = KT > 1 && kTiles > 1 ? KT : 1;          // items of a warp that are of one combination
+#pragma unroll
+      for (int i0 = 0; i0 < KT; i0 += kShare) {
+        const int combo = (KT * quad + i0) / kTiles;
+        float X[kShare][2][4];
+#pragma unroll
+        for (int i = 0; i < kShare; ++i)
+#pragma unroll
+          for (int e = 0; e < 2; ++e)
+#pragma unroll
+            for (int r = 0; r < 4; ++r) X[i][e][r] = 0.f;
+#pragma unroll
+        for (int s = 0; s < kTiles; ++s) {
+          const float4 fa = mail[(combo * NQ + 2 * s) * 32], fb = mail[(combo * NQ + 2 * s + 1) * 32];
+          unsigned hi[2][4], lo[2][4];
+          split_tf32(fa.x, hi[0][0], lo[0][0]);
+          split_tf32(fa.z, hi[0][1], lo[0][1]);
+          split_tf32(fb.x, hi[0][2], lo[0][2]);
+          split_tf32(fb.z, hi[0][3], lo[0][3]);
+          split_tf32(fa.y, hi[1][0], lo[1][0]);
+          split_tf32(fa.w, hi[1][1], lo[1][1]);
+          split_tf32(fb.y, hi[1][2], lo[1][2]);
+          split_tf32(fb.w, hi[1][3], lo[1][3]);
+#pragma unroll
+          for (int i = 0; i < kShare; ++i)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) mma_tf32(X[i][e], hi[e], T0[i0 + i][s], T1[i0 + i][s]);
+#pragma unroll
+          for (int i = 0; i < kShare; ++i)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) mma_tf32(X[i][e], lo[e], T0[i0 + i][s], T1[i0 + i][s]);
+        }
+        const int pair = combo & 1, key = key0 + (combo >> 1) * kTile + (lane >> 2);
+#pragma unroll
+        for (int i = 0; i < kShare; ++i) {
+#pragma unroll
+          for (int e = 0; e < 2; ++e)
+#pragma unroll
+            for (int r = 0; r < 4; ++r) {
+              float w = weight(X[i][e][r], p.neg_scale_log2, nb[i0 + i][r & 1]);
+              if (!full && (key + 8 * (r >> 1) > first_pos + 2 * pair + e || 2 * pair + e >= toks)) w = 0.f;
+              X[i][e][r] = w;
+            }
+          const int tile = (KT * quad + i0 + i) % kTiles;
+#pragma unroll
+          for (int u = 0; u < 2; ++u)
+            wmail[(combo * NQ + 2 * tile + u) * 32] = make_uint2(movmatrix_trans(pack_bf16(X[i][0][u], X[i][1][u])),
+                                                                 movmatrix_trans(pack_bf16(X[i][0][2 + u], X[i][1][2 + u])));
+        }
+      }
+    }
+    slot = slot + 1 == stages ? 0 : slot + 1;
+    arrive();                          // also: the weights are there
+    request();
+    if (compute) {
+      unsigned w0[KT][2], w1[KT][2];
 #pragma unroll
       for (int kt = 0; kt < KT; ++kt)
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
-          float X[2][4];
-#pragma unroll
-          for (int e = 0; e < 2; ++e)
-#pragma unroll
-            for (int r = 0; r < 4; ++r) X[e][r] = 0.f;
-#pragma unroll
-          for (int s = 0; s < NQ / 2; ++s) {
-            const float4 fa = mail[((kt * 2 + i) * NQ + 2 * s) * 32], fb = mail[((kt * 2 + i) * NQ + 2 * s + 1) * 32];
-            unsigned hi[4], lo[4];
-            split_tf32(fa.x, hi[0], lo[0]);
-            split_tf32(fa.z, hi[1], lo[1]);
-            split_tf32(fb.x, hi[2], lo[2]);
-            split_tf32(fb.z, hi[3], lo[3]);
-            mma_tf32(X[0], hi, T0[s], T1[s]);
-            mma_tf32(X[0], lo, T0[s], T1[s]);
-            split_tf32(fa.y, hi[0], lo[0]);
-            split_tf32(fa.w, hi[1], lo[1]);
-            split_tf32(fb.y, hi[2], lo[2]);
-            split_tf32(fb.w, hi[3], lo[3]);
-            mma_tf32(X[1], hi, T0[s], T1[s]);
-            mma_tf32(X[1], lo, T0[s], T1[s]);
-          }
-          float w[2][2];               // [token][key, key + 8]
-#pragma unroll
-          for (int e = 0; e < 2; ++e)
-#pragma unroll
-            for (int r = 0; r < 2; ++r) {
-              w[e][r] = weight(X[e][2 * r], p.neg_scale_log2, nb);
-              if (!full && (key0 + kt * kTile + (lane >> 2) + 8 * r > first_pos + 2 * i + e || 2 * i + e >= toks)) w[e][r] = 0.f;
-            }
-          w0[kt][i] = movmatrix_trans(pack_bf16(w[0][0], w[1][0]));
-          w1[kt][i] = movmatrix_trans(pack_bf16(w[0][1], w[1][1]));
+          const uint2 w = wmail[((kt * 2 + i) * NQ + quad) * 32];
+          w0[kt][i] = w.x, w1[kt][i] = w.y;
         }
-    }
-    slot = slot + 1 == stages ? 0 : slot + 1;
-    arrive();
-    request();
-    if (compute) {
       const unsigned base = ring_at + (unsigned)(slot * unit * 2);
       for (int c = c_first; c <= (ALIGNED ? c_first : c_last); ++c) {
         const unsigned head = base + (ALIGNED ? kv_off : c * HD * 2);
@@ -619,12 +657,11 @@ constexpr size_t kMaxSmem = 227 * 1024;
 int quads_for(int nq) { return nq <= 8 ? 2 : (nq <= 16 ? 4 : 8); }
 
 size_t tile_smem(int nkv, int hd, int kt, int stages) {
-  return (size_t)kTileWarps * 16 * hd * 2 + (size_t)kTileWarps * kt * 2 * 32 * 16 + (size_t)stages * kt * kTile * nkv * hd * 2;
+  return (size_t)kTileWarps * 16 * hd * 2 + (size_t)kTileWarps * kt * 2 * 32 * 24 + (size_t)stages * kt * kTile * nkv * hd * 2;
 }
 // key tiles of a step of the tile kernel and stages of its ring for a geometry: the most that fit (0: not two stages)
-int tile_stages(int nq, int nkv, int hd, int& kt) {
-  const bool aligned = (nq / nkv) % 4 == 0;
-  for (kt = 2; kt >= (aligned ? 2 : 1); --kt)
+int tile_stages(int nkv, int hd, int& kt) {
+  for (kt = 2; kt >= 1; --kt)
     for (int stages = 4; stages >= 2; --stages)
       if (tile_smem(nkv, hd, kt, stages) <= kMaxSmem) return stages;
   return 0;
@@ -639,14 +676,15 @@ size_t decode_smem(int nq, int hd) {
 template <int HD, int NQ>
 int launch_tiles(const SigParams& p, int items, cudaStream_t s) {
   int kt;
-  const int stages = tile_stages(p.nq, p.nkv, HD, kt);
+  const int stages = tile_stages(p.nkv, HD, kt);
   const size_t smem = tile_smem(p.nkv, HD, kt, stages);
 #define OI_SIG_TILE(KT, ALIGNED)                                                                                              \
   do {                                                                                                                        \
     OI_CHECK_CUDA(cudaFuncSetAttribute(sigmoid_tile_kernel<HD, NQ, KT, ALIGNED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kMaxSmem)); \
     oi_launch(sigmoid_tile_kernel<HD, NQ, KT, ALIGNED>, items, kTileWarps * 32, smem, s, p, stages);                          \
   } while (0)
-  if (p.group % 4 == 0) OI_SIG_TILE(2, true);
+  if (p.group % 4 == 0 && kt == 2) OI_SIG_TILE(2, true);
+  else if (p.group % 4 == 0) OI_SIG_TILE(1, true);
   else if (kt == 2) OI_SIG_TILE(2, false);
   else OI_SIG_TILE(1, false);
 #undef OI_SIG_TILE
@@ -687,7 +725,7 @@ bool aligned16(const void* p) { return ((uintptr_t)p & 15) == 0; }
 OI_API int oi_sigmoid_attention_tile_tokens(int nq, int nkv, int hd) {
   if ((hd != 32 && hd != 64 && hd != 128) || nq <= 0 || nkv <= 0 || nq % nkv || nq > 32) return 0;
   int kt;
-  return tile_stages(nq, nkv, hd, kt) > 0 && decode_smem(nq, hd) <= kMaxSmem ? 4 * (kTileWarps / quads_for(nq)) : 0;
+  return tile_stages(nkv, hd, kt) > 0 && decode_smem(nq, hd) <= kMaxSmem ? 4 * (kTileWarps / quads_for(nq)) : 0;
 }
 
 // bfloat16. Items: int32 [n, 4] (request, first token of the tile, slice, slices); a tile item covers

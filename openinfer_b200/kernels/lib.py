@@ -79,7 +79,7 @@ _SIGNATURES = {
     "oi_slice_sum_gate": [P, P, P, P, I, L, P, L, I, I, P],
     "oi_sigmoid_attention_tile_tokens": [I, I, I],
     "oi_sigmoid_attention_mma": [P, L, P, L, P, L, P, P, L, I, P, I, P, P, P, I, P, I, P, P, I, I, I, F, P, P, P],
-    "oi_mingru_scan": [P, I, L, P, L, I, P, P, L, P, P, P, I, I, I, I, P],
+    "oi_mingru_scan": [P, I, L, P, L, I, P, P, L, P, P, P, I, I, I, I, I, P],
     "oi_latent_rope_store": [P, L, I, I, P, L, I, I, I, I, P, I, F, F, I, P, P, I, P, P, I, I, I, I, P],
     "oi_add2_cast": [P, P, P, P, I, L, P],
     "oi_token_gate": [P, L, I, P, P, I, L, I, I, I, I, P],

@@ -856,5 +856,6 @@ def mingru_scan(out: torch.Tensor, zug: torch.Tensor, col_step: int, bias: torch
     _lib.check(_lib.load().oi_mingru_scan(
         out.data_ptr(), _code(out, "mingru_scan"), out.stride(0), zug.data_ptr(), zug.stride(0), int(col_step), bias.data_ptr(),
         state.data_ptr(), state.stride(0), ctx.cu_seqlens.data_ptr(), ctx.token_req.data_ptr(), ctx.state_slots.data_ptr(),
-        out.shape[0], ctx.num_requests, C, 1 if ctx.decode_only else 0, _stream()), "mingru_scan")
+        out.shape[0], ctx.num_requests, C, 1 if ctx.decode_only or 1 in ctx.q_lens_host else 0, 0 if ctx.decode_only else 1, _stream()),
+        "mingru_scan")
     return out

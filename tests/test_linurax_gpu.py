@@ -219,11 +219,11 @@ def test_scores_are_mixed_in_more_than_sixteen_bits():
 @pytest.mark.parametrize("channels", [1, 33, 64, 520])
 def test_gated_scan_kernel(channels, out_dtype):
     """Portions over old state beside a single token and a padding request; runs of rows that end inside a run, at a run's and
-    at a block's edge; the one-row kernel gives what the scan gives."""
+    at a round's edge."""
     from openinfer_b200.kernels import ops
     g = torch.Generator().manual_seed(channels)
     step = -(-channels // 8) * 8
-    for lens in ([7, 1, 128, 130], [1, 300], [1, 1, 1]):
+    for lens in ([7, 1, 256, 130], [1, 300], [2, 515, 5], [1, 1, 1]):
         T, B = sum(lens) + 1, len(lens) + 1
         zug = torch.randn(T, 3 * step, generator=g) * 2
         zug[0, :channels] = 40.0                          # an open gate forgets everything in front of it
@@ -236,10 +236,9 @@ def test_gated_scan_kernel(channels, out_dtype):
         class Ctx:
             cu_seqlens = _i32(starts)
             token_req = _i32([b for b, n in enumerate(lens) for _ in range(n)] + [-1])
-            state_slots, num_requests, decode_only = _i32(slots), B, False
+            state_slots, num_requests, decode_only, q_lens_host = _i32(slots), B, max(lens) == 1, lens + [1]
 
-        def run(decode_only=False):
-            Ctx.decode_only = decode_only
+        def run():
             y, s = torch.empty(T, channels, device="cuda", dtype=TORCH[out_dtype]), _dev(state.clone())
             ops.mingru_scan(y, _dev(zug), step, _dev(bias), s, Ctx)
             return y.double().cpu(), s.cpu()
@@ -255,10 +254,6 @@ def test_gated_scan_kernel(channels, out_dtype):
             assert (got - ref).abs().max().item() < (3e-6 if out_dtype == "float32" else 1e-2) * max(1.0, ref.abs().max().item())
             assert (s[slots[b]].double() - S[-1]).abs().max().item() < 3e-6 * max(1.0, S.abs().max().item())
         assert torch.equal(s[0], state[0]) and torch.equal(s[slots[-1]], state[slots[-1]])      # nobody's slot, and the padding's
-        if max(lens) == 1:
-            y1, s1 = run(decode_only=True)
-            assert torch.equal(y1[:-1], y[:-1]) or (y1[:-1] - y[:-1]).abs().max().item() < 1e-6
-            assert (s1 - s).abs().max().item() < 1e-6
 
 
 # ---------------------------------------------------------------------------------------------- mechanisms alone
