@@ -230,11 +230,7 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) sigmoid_tile_kernel(const 
     rq_slot = rq_slot + 1 == stages ? 0 : rq_slot + 1;
     cp_async_commit();
   };
-  auto arrive = [&]() {                // the oldest stage requested is there, and every warp is done with the one before it
-    if (stages == 4) cp_async_wait<2>(); else if (stages == 3) cp_async_wait<1>(); else cp_async_wait<0>();
-    __syncthreads();
-  };
-  for (int u = 0; u < stages - 1; ++u) request();
+  for (int u = 0; u < stages; ++u) request();
 
   for (int i = lane; i < 16 * head_chunks; i += 32) {
     const int r = i / head_chunks, ch = i % head_chunks;
@@ -292,145 +288,164 @@ __global__ void __launch_bounds__(kTileWarps * 32, 1) sigmoid_tile_kernel(const 
   const unsigned ring_at = smem_u32(ring);
   const int tile_bytes = kTile * row_elems * 2;
 
-  int slot = 0;
-  for (int u = 0; u < units; u += 2) {
-    const int key0 = (t_begin + (u >> 1)) * kStep;
-    const bool compute = key0 <= last_pos;          // the same for all warps of four tokens
-    arrive();
-    request();
-    if (compute) {
-      float S[KT][2][4];
+  // The raw scores of a step out of its K, left for the warps that mix them.
+  auto form_scores = [&](int slot) {
+    float S[KT][2][4];
 #pragma unroll
-      for (int kt = 0; kt < KT; ++kt)
+    for (int kt = 0; kt < KT; ++kt)
 #pragma unroll
-        for (int i = 0; i < 2; ++i)
+      for (int i = 0; i < 2; ++i)
 #pragma unroll
-          for (int e = 0; e < 4; ++e) S[kt][i][e] = 0.f;
-      const unsigned base = ring_at + (unsigned)(slot * unit * 2);
-      for (int c = c_first; c <= (ALIGNED ? c_first : c_last); ++c) {
-        const unsigned head = base + (ALIGNED ? kv_off : c * HD * 2);
-        bool mine = true;
-        if constexpr (!ALIGNED) {
-          const int h = 4 * quad + (lane >> 3);
-          mine = h >= c * p.group && h < (c + 1) * p.group;
-        }
-#pragma unroll
-        for (int k2 = 0; k2 < HD / 32; ++k2) {
-          unsigned b[2][4], a[KT][2][4];
-#pragma unroll
-          for (int kt = 0; kt < KT; ++kt)
-#pragma unroll
-            for (int x = 0; x < 2; ++x)
-              ldmatrix_x4(a[kt][x], head + kt * tile_bytes + k_at[(2 * k2 + x) % kJ] + ((2 * k2 + x) / 4) * 128);
-#pragma unroll
-          for (int i = 0; i < 2; ++i) {
-            ldmatrix_x4(b[i], q_at[k2 & 1] + i * 8 * HD * 2 + (k2 >> 1) * 128);
-            if constexpr (!ALIGNED) {
-#pragma unroll
-              for (int r = 0; r < 4; ++r) b[i][r] = mine ? b[i][r] : 0u;
-            }
-          }
-#pragma unroll
-          for (int x = 0; x < 2; ++x)
-#pragma unroll
-            for (int kt = 0; kt < KT; ++kt)
-#pragma unroll
-              for (int i = 0; i < 2; ++i) mma_bf16(S[kt][i], a[kt][x], b[i][2 * x], b[i][2 * x + 1]);
-        }
+        for (int e = 0; e < 4; ++e) S[kt][i][e] = 0.f;
+    const unsigned base = ring_at + (unsigned)(slot * unit * 2);
+    for (int c = c_first; c <= (ALIGNED ? c_first : c_last); ++c) {
+      const unsigned head = base + (ALIGNED ? kv_off : c * HD * 2);
+      bool mine = true;
+      if constexpr (!ALIGNED) {
+        const int h = 4 * quad + (lane >> 3);
+        mine = h >= c * p.group && h < (c + 1) * p.group;
       }
-      // (everyone has read the last step's scores: two barriers of the block lie between; the weights likewise)
 #pragma unroll
-      for (int kt = 0; kt < KT; ++kt)
-#pragma unroll
-        for (int i = 0; i < 2; ++i) mail[((kt * 2 + i) * NQ + quad) * 32] = make_float4(S[kt][i][0], S[kt][i][1], S[kt][i][2], S[kt][i][3]);
-      asm volatile("bar.sync %0, %1;\n" ::"r"(group4 + 1), "n"(NQ * 32) : "memory");
-      const bool full = key0 + kStep - 1 <= first_pos && toks == 4;
-      constexpr int kShare = KT > 1 && kTiles > 1 ? KT : 1;          // items of a warp that are of one combination
-#pragma unroll
-      for (int i0 = 0; i0 < KT; i0 += kShare) {
-        const int combo = (KT * quad + i0) / kTiles;
-        float X[kShare][2][4];
-#pragma unroll
-        for (int i = 0; i < kShare; ++i)
-#pragma unroll
-          for (int e = 0; e < 2; ++e)
-#pragma unroll
-            for (int r = 0; r < 4; ++r) X[i][e][r] = 0.f;
-#pragma unroll
-        for (int s = 0; s < kTiles; ++s) {
-          const float4 fa = mail[(combo * NQ + 2 * s) * 32], fb = mail[(combo * NQ + 2 * s + 1) * 32];
-          unsigned hi[2][4], lo[2][4];
-          split_tf32(fa.x, hi[0][0], lo[0][0]);
-          split_tf32(fa.z, hi[0][1], lo[0][1]);
-          split_tf32(fb.x, hi[0][2], lo[0][2]);
-          split_tf32(fb.z, hi[0][3], lo[0][3]);
-          split_tf32(fa.y, hi[1][0], lo[1][0]);
-          split_tf32(fa.w, hi[1][1], lo[1][1]);
-          split_tf32(fb.y, hi[1][2], lo[1][2]);
-          split_tf32(fb.w, hi[1][3], lo[1][3]);
-#pragma unroll
-          for (int i = 0; i < kShare; ++i)
-#pragma unroll
-            for (int e = 0; e < 2; ++e) mma_tf32(X[i][e], hi[e], T0[i0 + i][s], T1[i0 + i][s]);
-#pragma unroll
-          for (int i = 0; i < kShare; ++i)
-#pragma unroll
-            for (int e = 0; e < 2; ++e) mma_tf32(X[i][e], lo[e], T0[i0 + i][s], T1[i0 + i][s]);
-        }
-        const int pair = combo & 1, key = key0 + (combo >> 1) * kTile + (lane >> 2);
-#pragma unroll
-        for (int i = 0; i < kShare; ++i) {
-#pragma unroll
-          for (int e = 0; e < 2; ++e)
-#pragma unroll
-            for (int r = 0; r < 4; ++r) {
-              float w = weight(X[i][e][r], p.neg_scale_log2, nb[i0 + i][r & 1]);
-              if (!full && (key + 8 * (r >> 1) > first_pos + 2 * pair + e || 2 * pair + e >= toks)) w = 0.f;
-              X[i][e][r] = w;
-            }
-          const int tile = (KT * quad + i0 + i) % kTiles;
-#pragma unroll
-          for (int u = 0; u < 2; ++u)
-            wmail[(combo * NQ + 2 * tile + u) * 32] = make_uint2(movmatrix_trans(pack_bf16(X[i][0][u], X[i][1][u])),
-                                                                 movmatrix_trans(pack_bf16(X[i][0][2 + u], X[i][1][2 + u])));
-        }
-      }
-    }
-    slot = slot + 1 == stages ? 0 : slot + 1;
-    arrive();                          // also: the weights are there
-    request();
-    if (compute) {
-      unsigned w0[KT][2], w1[KT][2];
-#pragma unroll
-      for (int kt = 0; kt < KT; ++kt)
-#pragma unroll
-        for (int i = 0; i < 2; ++i) {
-          const uint2 w = wmail[((kt * 2 + i) * NQ + quad) * 32];
-          w0[kt][i] = w.x, w1[kt][i] = w.y;
-        }
-      const unsigned base = ring_at + (unsigned)(slot * unit * 2);
-      for (int c = c_first; c <= (ALIGNED ? c_first : c_last); ++c) {
-        const unsigned head = base + (ALIGNED ? kv_off : c * HD * 2);
-        bool mine = true;
-        if constexpr (!ALIGNED) {
-          const int h = 4 * quad + (lane >> 3);
-          mine = h >= c * p.group && h < (c + 1) * p.group;
-        }
+      for (int k2 = 0; k2 < HD / 32; ++k2) {
+        unsigned b[2][4], a[KT][2][4];
 #pragma unroll
         for (int kt = 0; kt < KT; ++kt)
 #pragma unroll
-          for (int m2 = 0; m2 < HD / 16; m2 += 2) {
-            unsigned a[2][4];
+          for (int x = 0; x < 2; ++x)
+            ldmatrix_x4(a[kt][x], head + kt * tile_bytes + k_at[(2 * k2 + x) % kJ] + ((2 * k2 + x) / 4) * 128);
 #pragma unroll
-            for (int x = 0; x < 2; ++x) ldmatrix_x4_trans(a[x], head + kt * tile_bytes + v_at[(m2 + x) % kJ] + ((m2 + x) / 4) * 128);
+        for (int i = 0; i < 2; ++i) {
+          ldmatrix_x4(b[i], q_at[k2 & 1] + i * 8 * HD * 2 + (k2 >> 1) * 128);
+          if constexpr (!ALIGNED) {
 #pragma unroll
-            for (int x = 0; x < 2; ++x)
-#pragma unroll
-              for (int i = 0; i < 2; ++i) mma_bf16(O[i][m2 + x], a[x], mine ? w0[kt][i] : 0u, mine ? w1[kt][i] : 0u);
+            for (int r = 0; r < 4; ++r) b[i][r] = mine ? b[i][r] : 0u;
           }
+        }
+#pragma unroll
+        for (int x = 0; x < 2; ++x)
+#pragma unroll
+          for (int kt = 0; kt < KT; ++kt)
+#pragma unroll
+            for (int i = 0; i < 2; ++i) mma_bf16(S[kt][i], a[kt][x], b[i][2 * x], b[i][2 * x + 1]);
       }
     }
-    slot = slot + 1 == stages ? 0 : slot + 1;
+#pragma unroll
+    for (int kt = 0; kt < KT; ++kt)
+#pragma unroll
+      for (int i = 0; i < 2; ++i) mail[((kt * 2 + i) * NQ + quad) * 32] = make_float4(S[kt][i][0], S[kt][i][1], S[kt][i][2], S[kt][i][3]);
+  };
+  // This warp's share of a step's mix and weights, left for the warps that own the heads.
+  auto form_weights = [&](int key0) {
+    const bool full = key0 + kStep - 1 <= first_pos && toks == 4;
+    constexpr int kShare = KT > 1 && kTiles > 1 ? KT : 1;          // items of a warp that are of one combination
+#pragma unroll
+    for (int i0 = 0; i0 < KT; i0 += kShare) {
+      const int combo = (KT * quad + i0) / kTiles;
+      float X[kShare][2][4];
+#pragma unroll
+      for (int i = 0; i < kShare; ++i)
+#pragma unroll
+        for (int e = 0; e < 2; ++e)
+#pragma unroll
+          for (int r = 0; r < 4; ++r) X[i][e][r] = 0.f;
+#pragma unroll
+      for (int s = 0; s < kTiles; ++s) {
+        const float4 fa = mail[(combo * NQ + 2 * s) * 32], fb = mail[(combo * NQ + 2 * s + 1) * 32];
+        unsigned hi[2][4], lo[2][4];
+        split_tf32(fa.x, hi[0][0], lo[0][0]);
+        split_tf32(fa.z, hi[0][1], lo[0][1]);
+        split_tf32(fb.x, hi[0][2], lo[0][2]);
+        split_tf32(fb.z, hi[0][3], lo[0][3]);
+        split_tf32(fa.y, hi[1][0], lo[1][0]);
+        split_tf32(fa.w, hi[1][1], lo[1][1]);
+        split_tf32(fb.y, hi[1][2], lo[1][2]);
+        split_tf32(fb.w, hi[1][3], lo[1][3]);
+#pragma unroll
+        for (int i = 0; i < kShare; ++i)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) mma_tf32(X[i][e], hi[e], T0[i0 + i][s], T1[i0 + i][s]);
+#pragma unroll
+        for (int i = 0; i < kShare; ++i)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) mma_tf32(X[i][e], lo[e], T0[i0 + i][s], T1[i0 + i][s]);
+      }
+      const int pair = combo & 1, key = key0 + (combo >> 1) * kTile + (lane >> 2);
+#pragma unroll
+      for (int i = 0; i < kShare; ++i) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e)
+#pragma unroll
+          for (int r = 0; r < 4; ++r) {
+            float w = weight(X[i][e][r], p.neg_scale_log2, nb[i0 + i][r & 1]);
+            if (!full && (key + 8 * (r >> 1) > first_pos + 2 * pair + e || 2 * pair + e >= toks)) w = 0.f;
+            X[i][e][r] = w;
+          }
+        const int tile = (KT * quad + i0 + i) % kTiles;
+#pragma unroll
+        for (int u = 0; u < 2; ++u)
+          wmail[(combo * NQ + 2 * tile + u) * 32] = make_uint2(movmatrix_trans(pack_bf16(X[i][0][u], X[i][1][u])),
+                                                               movmatrix_trans(pack_bf16(X[i][0][2 + u], X[i][1][2 + u])));
+      }
+    }
+  };
+  // The step's weights (this warp's heads) times its V.
+  auto add_values = [&](int slot) {
+    unsigned w0[KT][2], w1[KT][2];
+#pragma unroll
+    for (int kt = 0; kt < KT; ++kt)
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const uint2 w = wmail[((kt * 2 + i) * NQ + quad) * 32];
+        w0[kt][i] = w.x, w1[kt][i] = w.y;
+      }
+    const unsigned base = ring_at + (unsigned)(slot * unit * 2);
+    for (int c = c_first; c <= (ALIGNED ? c_first : c_last); ++c) {
+      const unsigned head = base + (ALIGNED ? kv_off : c * HD * 2);
+      bool mine = true;
+      if constexpr (!ALIGNED) {
+        const int h = 4 * quad + (lane >> 3);
+        mine = h >= c * p.group && h < (c + 1) * p.group;
+      }
+#pragma unroll
+      for (int kt = 0; kt < KT; ++kt)
+#pragma unroll
+        for (int m2 = 0; m2 < HD / 16; m2 += 2) {
+          unsigned a[2][4];
+#pragma unroll
+          for (int x = 0; x < 2; ++x) ldmatrix_x4_trans(a[x], head + kt * tile_bytes + v_at[(m2 + x) % kJ] + ((m2 + x) / 4) * 128);
+#pragma unroll
+          for (int x = 0; x < 2; ++x)
+#pragma unroll
+            for (int i = 0; i < 2; ++i) mma_bf16(O[i][m2 + x], a[x], mine ? w0[kt][i] : 0u, mine ? w1[kt][i] : 0u);
+        }
+    }
+  };
+  // Two meetings of the block a step. Between the first and the second: the values of a step and the raw scores of the next
+  // one, which do not wait for one another; between the second and the next first: that step's mix. So scores are read, and
+  // weights written, while nobody writes scores or reads weights.
+  const int steps = units / 2;
+  auto seen = [&](int n) { return n < steps && (t_begin + n) * kStep <= last_pos; };      // the same for all warps of four tokens
+  auto next_slot = [&](int slot) { return slot + 1 == stages ? 0 : slot + 1; };
+  if (steps > 0) {
+    if (stages == 4) cp_async_wait<3>(); else if (stages == 3) cp_async_wait<2>(); else cp_async_wait<1>();
+    __syncthreads();
+    if (seen(0)) form_scores(0);
+    __syncthreads();
+    request();
+    if (seen(0)) form_weights(t_begin * kStep);
+  }
+  int slot = 1;
+  for (int n = 0; n < steps; ++n) {
+    if (stages == 4) cp_async_wait<2>(); else if (stages == 3) cp_async_wait<1>(); else cp_async_wait<0>();
+    __syncthreads();
+    const int k_slot = next_slot(slot);
+    if (seen(n)) add_values(slot);
+    if (seen(n + 1)) form_scores(k_slot);
+    __syncthreads();
+    request();
+    request();
+    if (seen(n + 1)) form_weights((t_begin + n + 1) * kStep);
+    slot = next_slot(k_slot);
   }
   cp_async_wait<0>();
 

@@ -20,6 +20,8 @@ from .attention import _sm_count
 PAGE_MULTIPLE = 16
 KEYS_PER_STEP = 32
 MIN_STEPS_PER_SLICE = 8         # a prompt tile's slice is at least 256 keys long
+SLICE_SHARE = 0.65              # of an even share of all tiles' keys over the SMs: the longest slice, where there are no more
+                                # tiles than SMs (prompts of 1,024 to 4,096 tokens: 5-15 % shorter than a whole share)
 DECODE_MIN_KEYS_PER_SLICE = 64  # a step of 16 keys for each of the CTA's four warps
 DECODE_MAX_SLICES = 64
 DECODE_CTAS_PER_SM = 2
@@ -50,7 +52,7 @@ def plan_items(q_lens: Sequence[int], kv_lens: Sequence[int], tile_tokens: int, 
                fixed_decode_slices: Optional[int] = None):
     """Work items of one step: (tile_items [n, 4], decode_items [n, 4], row_splits [tokens], row_base [tokens], partial rows).
 
-    A prompt tile's keys are cut so that no item is longer than (three quarters of) an even share of all tiles' keys over the
+    A prompt tile's keys are cut so that no item is longer than (SLICE_SHARE of) an even share of all tiles' keys over the
     SMs, or MIN_STEPS_PER_SLICE steps: the last tiles of a long prompt would otherwise still run when the others are done."""
     starts = np.concatenate([[0], np.cumsum(q_lens)]).astype(np.int64)
     tokens = int(starts[-1])
@@ -72,7 +74,7 @@ def plan_items(q_lens: Sequence[int], kv_lens: Sequence[int], tile_tokens: int, 
     limit = None
     if tiles and not policy.batch_invariant():
         share = sum(t[3] for t in tiles) / sm_count
-        limit = max(MIN_STEPS_PER_SLICE, int((0.75 if len(tiles) < 2 * sm_count else 1.0) * share) + 1)
+        limit = max(MIN_STEPS_PER_SLICE, int((SLICE_SHARE if len(tiles) <= sm_count else 1.0) * share) + 1)
     items = []
     for b, t0, toks, steps in tiles:
         ns = -(-steps // limit) if limit else 1
