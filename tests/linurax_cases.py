@@ -45,7 +45,7 @@ CASE_B = model(97, 48, [
 ], eps=1e-6, scale=1.0)
 # heads the tensor-core kernels take in bfloat16, one group size each
 CASE_C = model(300, 128, [
-    attn(6, 2, 32, 0.3, rot=(16, 20000.0), mlp=96), gru(256, mlp=64), attn(8, 2, 64, 0.25, rot=(64, 10000.0)),
+    attn(6, 2, 32, 0.3, rot=(16, 30000.0), mlp=96), gru(256, mlp=64), attn(8, 2, 64, 0.25, rot=(64, 10000.0)),
     attn(16, 2, 64, 0.2, rot=(32, 500.0), mlp=160), attn(2, 1, 128, 0.15, rot=(128, 1000000.0)), gru(33), attn(20, 5, 32, 0.35, rot=(30, 100.0)),
 ], eps=1e-6, scale=0.7)
 # sizes that are multiples of nothing

@@ -59,7 +59,7 @@ def save(path, tensors):
 # ---------------------------------------------------------------------------------------------- kernels alone
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("nq,nkv,hd,qk,rot_half,own_values,page", [(4, 2, 16, 16, 4, False, 16), (3, 1, 16, 10, 3, False, 4),
-                                                                    (5, 5, 40, 40, 0, False, 8), (6, 2, 64, 64, 32, True, 16),
+                                                                    (5, 5, 40, 40, 0, False, 8), (9, 3, 64, 64, 32, True, 16),
                                                                     (1, 1, 8, 6, 1, False, 2), (20, 5, 128, 128, 64, False, 16)])
 def test_joint_norm_rotation_and_store_kernel(dtype, nq, nkv, hd, qk, rot_half, own_values, page):
     """q and k normed over all heads together, neighbouring pairs turned, q in place, k to its page, and as the value the key
@@ -146,7 +146,7 @@ def _attention_case(nq, nkv, hd, q_lens, kv_lens, page, td, seed):
 
 
 @pytest.mark.parametrize("tensor_cores", [True, False])
-@pytest.mark.parametrize("nq,nkv,hd", [(6, 2, 64), (4, 1, 32), (8, 8, 64), (16, 4, 128), (12, 4, 64), (32, 8, 128), (20, 5, 32), (3, 3, 128),
+@pytest.mark.parametrize("nq,nkv,hd", [(9, 3, 64), (4, 1, 32), (8, 8, 64), (16, 4, 128), (12, 4, 64), (32, 8, 128), (20, 5, 32), (3, 3, 128),
                                        (1, 1, 64), (16, 16, 128), (24, 2, 32), (5, 1, 24), (2, 2, 256)])
 def test_attention_kernels_over_paged_keys(nq, nkv, hd, tensor_cores):
     """The tensor-core kernels and the general one, on shuffled pages: prompt portions behind cached keys beside single tokens,
@@ -425,7 +425,7 @@ def _sharp_model(tmp_path, name, heads, dim, rot=None, seed=11):
     return cfg, path
 
 
-@pytest.mark.parametrize("heads,dim,rot", [((4, 2), 16, (4, 10000.0)), ((6, 2), 64, (8, 10000.0)), ((4, 1), 32, None)])
+@pytest.mark.parametrize("heads,dim,rot", [((4, 2), 16, (4, 10000.0)), ((9, 3), 64, (8, 10000.0)), ((4, 1), 32, None)])
 def test_far_keys_first_tokens_and_keys_at_borders(tmp_path, heads, dim, rot):
     """A row's result rests on the few keys that match it, wherever they are among 400: in prompts, in portions and decoded.
     The comparison is sharp: the plain implementation with one key taken away, the first, the ones at the edges of pages and of
