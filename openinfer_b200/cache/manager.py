@@ -2,7 +2,7 @@
 layers that share a geometry, and slots for per-request state of fixed size.
 
 A *group* is the set of layers (more exactly: of calls in the model's run order)
-whose mixers asked for the same (kv heads, head size, window). Each group has a
+whose mixers asked for the same (kv heads, head size, window or chunk). Each group has a
 pool of pages of its own; a page id names ``page_size`` positions of every layer of
 the group, K and V. The device tensor is laid out layer first,
 ``[layers_in_group, 2, pages, page_size, kv_heads, head_dim]``: what one layer's
@@ -11,8 +11,8 @@ instead of being strewn over the whole pool at a stride of one page of all layer
 the reference's page-first buffer (pegainfer-kv-cache/src/layout.rs:5-33), which keeps
 the address translation and the DRAM rows of a layer's pass local. A request holds, per group, a block table:
 page ids in position order. Pages go back to the pool when the request ends, or,
-in a group with a window, as soon as every position of the page is further back
-than the window of any query still to come.
+in a group with a window (or chunks), as soon as every position of the page is further back
+than the window (or chunk) of any query still to come.
 
 Prefix cache (optional; the reference's is on by default, kvbm-logical scheduled.rs:436-459): a FULL
 page of PROMPT tokens is registered under a lineage key, the digest of (its parent's key, its token ids).
@@ -49,6 +49,7 @@ class KvNeed:
     head_dim: int
     window: Optional[int] = None  # keys a query sees, itself included; None = all
     planes: int = 2               # 2: keys and values; 1: one tensor per position that serves as both (a latent)
+    chunked: bool = False         # ``window`` is a chunk's size: a query sees the keys of its own chunk, counted from position 0
     keep_first: int = 0           # with a window: the first positions of a sequence that stay visible behind it (their pages stay)
 
 
@@ -208,7 +209,7 @@ class CacheManager:
         """Lowest page index a query at position >= start can read in group g."""
         if g.window is None:
             return 0
-        first_key = max(0, start - g.window + 1)
+        first_key = start - start % g.window if g.need.chunked else max(0, start - g.window + 1)
         return first_key // self.page_size
 
     def pages_needed(self, request_id: Hashable, new_tokens: int) -> List[int]:

@@ -16,9 +16,11 @@ from .linurax import LinuraxConfig
 from .luzitar import LuzitarConfig
 from .pilonex import PilonexConfig
 from .qwen3 import Qwen3Config
+from .rolevik import RolevikConfig
 
 __all__ = [
-    "ArchitectureEntry", "BubalixConfig", "ConfigError", "DelunexConfig", "LinuraxConfig", "LuzitarConfig", "ModelConfig", "PilonexConfig", "Qwen3Config", "known_architectures",
+    "ArchitectureEntry", "BubalixConfig", "ConfigError", "DelunexConfig", "LinuraxConfig", "LuzitarConfig", "ModelConfig", "PilonexConfig",
+    "Qwen3Config", "RolevikConfig", "known_architectures",
     "load_config", "read_config_json", "register_architecture", "resolve_architecture",
     "unregister_architecture",
 ]

@@ -1,8 +1,8 @@
 // Paged causal attention, general form: any head_dim that is a multiple of 8 (up to 512), any
-// number of heads and groups, an optional window, float32 or bfloat16 storage; prompt portions
+// number of heads and groups, an optional window or chunks, float32 or bfloat16 storage; prompt portions
 // and single decoded tokens alike. One warp per (token, query head).
 //
-// s[i,j] = (q_i . k_j) * scale for j <= pos_i (and j > pos_i - window, or j among the sequence's kept first keys),
+// s[i,j] = (q_i . k_j) * scale for first_visible(pos_i) <= j <= pos_i (and j among the sequence's kept first keys),
 // online softmax in float32,
 // o_i = sum_j p[i,j] v_j; query head h reads kv head h / (nq / nkv)
 // (pegainfer-kernels/csrc/shared/paged_attention.cu:439-567; pegainfer-kernels/src/ops/attention.rs:507).
@@ -66,7 +66,7 @@ __global__ void attention_generic_kernel(
   for (int d = lane; d < hd; d += 32) q_sh[warp][d] = to_f32(qp[d]);
   __syncwarp();
 
-  const int first = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+  const int first = first_visible(pos, window);
   const size_t row_elems = (size_t)nkv * hd;
   constexpr int VN = Vec16<T>::N;
   constexpr int kAccs = kMaxHd / 32;

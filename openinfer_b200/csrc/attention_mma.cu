@@ -10,7 +10,7 @@
 // pegainfer-kernels/csrc/shared/paged_attention.cu:189-263), in which case it writes a normalised
 // partial output and its log-sum-exp to scratch and `attention_merge_kernel` combines the slices.
 //
-// Math: s = (q . k) / sqrt(hd) for keys j <= pos (and j > pos - window), online softmax in float32
+// Math: s = (q . k) / sqrt(hd) for keys first_visible(pos) <= j <= pos (a window or chunks), online softmax in float32
 // (exp2 with the scale folded in), o = sum p v (paged_attention.cu:439-567). K/V tiles of 64 keys
 // are gathered page by page with cp.async into swizzled shared memory, double buffered;
 // S = Q K^T and O = P V run as mma.sync m16n8k16 with float32 accumulators.
@@ -35,7 +35,7 @@ struct AttnParams {
   const int4* items;       // (request, first token of the tile, split, nsplits)
   int nq, nkv, group;
   float scale_log2;        // softmax scale * log2(e)
-  int window;              // 0 = none
+  int window;              // 0: every key; > 0: the last `window` keys; < 0: the keys of the query's chunk of -window positions
   float* part_o; float* part_lse; int max_splits;  // scratch for split items
   int merge_in_kernel;     // decode kernel: the CTAs of a row form a cluster and merge their slices themselves:
                            // 1 by reading each other's shared memory, 2 by depositing partials with the merging CTA
@@ -149,8 +149,7 @@ attention_mma_kernel(const AttnParams p) {
   const int tile_toks = min(toks_per_tile, q_len - tok0);
   const int pos0 = kv_len - q_len + tok0;                 // position of the tile's first token
   // keys any row of the tile may see
-  int lo = 0;
-  if (p.window > 0) lo = max(0, pos0 - p.window + 1);
+  int lo = first_visible(pos0, p.window);
   const int hi = pos0 + tile_toks;                        // exclusive: last token's own key included
   lo &= ~(kKeys - 1);
   // a window that keeps the sequence's first keys visible: the tiles that hold them come first in the item's list of
@@ -180,7 +179,7 @@ attention_mma_kernel(const AttnParams p) {
 
   // ---- the rows this thread owns: slab mt, halves i: row = warp*16*MT + mt*16 + lane/4 + 8*i
   const int warp_row0 = warp * 16 * MT;
-  int pos[MT][2];
+  int pos[MT][2], first[MT][2];       // the row's position and the first key it sees
   bool row_ok[MT][2];
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
@@ -190,10 +189,12 @@ attention_mma_kernel(const AttnParams p) {
       const int t = r / group;
       row_ok[mt][i] = t < tile_toks;
       pos[mt][i] = pos0 + t;
+      first[mt][i] = first_visible(pos0 + t, p.window);
     }
   // the last position any row of this warp holds: tiles beyond it are skipped by this warp
   const int warp_last_pos = pos0 + min(tile_toks - 1, (warp_row0 + 16 * MT - 1) / group);
   const int warp_first_pos = pos0 + warp_row0 / group;
+  const int warp_last_first = first_visible(warp_last_pos, p.window);   // every row of the warp sees the keys from here on
   const bool warp_active = warp_row0 < tile_toks * group;
 
   constexpr int kSteps = HD / 16;
@@ -301,7 +302,7 @@ attention_mma_kernel(const AttnParams p) {
       }
       // ---- mask (only where a row may not see the whole tile) + online softmax
       const bool full = key0 + kKeys - 1 <= warp_first_pos &&
-                        (p.window <= 0 || key0 > warp_last_pos - p.window || key0 + kKeys <= keep_first) &&
+                        (key0 >= warp_last_first || key0 + kKeys <= keep_first) &&
                         warp_row0 + 16 * MT <= tile_toks * group;
       if (MODS) {
 #pragma unroll
@@ -332,7 +333,7 @@ attention_mma_kernel(const AttnParams p) {
               const int i = e >> 1;
               const int key = key0 + j * 8 + (lane & 3) * 2 + (e & 1);
               const bool ok = row_ok[mt][i] && key <= pos[mt][i] &&
-                              (p.window <= 0 || key > pos[mt][i] - p.window || key < keep_first);
+                              (key >= first[mt][i] || key < keep_first);
               s[mt][j][e] = ok ? s[mt][j][e] : -INFINITY;
               m_new[i] = fmaxf(m_new[i], s[mt][j][e]);
             }
@@ -583,8 +584,8 @@ attention_decode_kernel(const AttnParams p) {
   const int kv_len = p.kv_lens[req];
   const int* bt = p.block_table + (size_t)req * p.bt_stride;
   const int pos = kv_len - 1;
-  int lo = 0;
-  if (p.window > 0) lo = max(0, pos - p.window + 1) & ~(kDecKeys - 1);
+  const int first = first_visible(pos, p.window);
+  const int lo = first & ~(kDecKeys - 1);
   // a window that keeps the sequence's first keys visible: their tiles come first in the row's list of tiles, as far as
   // they lie wholly in front of the window's
   const int keep_first = (MODS && p.window > 0) ? p.mods.keep_first : 0;
@@ -773,7 +774,7 @@ attention_decode_kernel(const AttnParams p) {
       float m_new[2] = {m[0], m[1]};
       // a tile whose every key every row sees needs no mask (rows beyond the group hold zeros
       // and are never stored)
-      const bool full = key0 + kDecKeys <= kv_len && (p.window <= 0 || key0 > pos - p.window || key0 + kDecKeys <= keep_first);
+      const bool full = key0 + kDecKeys <= kv_len && (key0 >= first || key0 + kDecKeys <= keep_first);
       const float sl2 = MODS ? 1.f : p.scale_log2;
       if (MODS) {
 #pragma unroll
@@ -798,7 +799,7 @@ attention_decode_kernel(const AttnParams p) {
           for (int e = 0; e < 4; ++e) {
             const int i = e >> 1;
             const int key = key0 + j * 8 + (lane & 3) * 2 + (e & 1);
-            const bool ok = key <= pos && (p.window <= 0 || key > pos - p.window || key < keep_first);
+            const bool ok = key <= pos && (key >= first || key < keep_first);
             s[j][e] = ok ? s[j][e] * sl2 : -INFINITY;
             m_new[i] = fmaxf(m_new[i], s[j][e]);
           }

@@ -30,7 +30,7 @@
 // and a flag that ends all roles, after which the CTA frees its tensor memory and returns.
 // No load uses cluster multicast.
 //
-// Math as the other attention kernels: s = (q . k) / sqrt(hd) for keys j <= pos (and j > pos - window),
+// Math as the other attention kernels: s = (q . k) / sqrt(hd) for keys first_visible(pos) <= j <= pos (a window or chunks),
 // softmax in float32 with exp2 and the scale folded in, o = sum p v
 // (pegainfer-kernels/csrc/shared/paged_attention.cu:439-567).
 #include "oi_api.h"
@@ -139,9 +139,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
   const int toks_per_tile = kRows / group;
   const int tile_toks = min(toks_per_tile, q_len - tok0);
   const int pos0 = kv_len - q_len + tok0;
-  int lo = 0;
-  if (p.window > 0) lo = max(0, pos0 - p.window + 1);
-  lo &= ~(kKeys - 1);
+  int lo = first_visible(pos0, p.window) & ~(kKeys - 1);
   const int hi = pos0 + tile_toks;
   // An item may cover a slice of the tile's keys (when whole tiles would leave SMs idle): key tiles
   // [t_begin, t_end) of the span, cut as in the mma.sync kernel; its result goes to scratch, normalised and with
@@ -291,6 +289,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     const int t_row = r / group;
     const bool row_ok = t_row < tile_toks;
     const int pos = pos0 + t_row;
+    const int first = first_visible(pos, p.window);     // the first key this row sees
     const unsigned lane_base = tmem + ((unsigned)(quarter * 32) << 16);
     float m_ref = -INFINITY;                            // the maximum P is taken relative to (raw score units)
     float l = 0.f;
@@ -310,12 +309,12 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
 #pragma unroll
         for (int e = 0; e < 32; ++e) { sv[e] = __uint_as_float(v0[e]); sv[32 + e] = __uint_as_float(v1[e]); }
       }
-      const bool full = row_ok && key0 + kKeys - 1 <= pos && (p.window <= 0 || key0 > pos - p.window);
+      const bool full = row_ok && key0 + kKeys - 1 <= pos && key0 >= first;
       if (!full) {
 #pragma unroll
         for (int e = 0; e < kKeys; ++e) {
           const int key = key0 + e;
-          const bool vis = row_ok && key <= pos && (p.window <= 0 || key > pos - p.window);
+          const bool vis = row_ok && key <= pos && key >= first;
           sv[e] = vis ? sv[e] : -INFINITY;
         }
       }

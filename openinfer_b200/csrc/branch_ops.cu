@@ -19,8 +19,9 @@ __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + lo
 
 // ---------------------------------------------------------------------------------------------
 // out[r] = round( x[src] * rsqrt(mean(x[src]^2) + eps) * (w_offset + w) ), src = row_idx ? row_idx[r] : r
+// kCenter (a layer norm): the row's mean is taken off first
 // ---------------------------------------------------------------------------------------------
-template <typename TX, typename TO>
+template <typename TX, typename TO, bool kCenter>
 __global__ void rmsnorm_cast_kernel(TO* __restrict__ out, const TX* __restrict__ x, const void* __restrict__ w, int w_dtype,
                                     const int* __restrict__ row_idx, int hidden, float eps, float w_offset) {
   pdl_start();
@@ -28,16 +29,21 @@ __global__ void rmsnorm_cast_kernel(TO* __restrict__ out, const TX* __restrict__
   const int r = blockIdx.x;
   const size_t src = row_idx ? (size_t)row_idx[r] : (size_t)r;
   const TX* xr = x + src * hidden;
+  float mean = 0.f;
+  if (kCenter) {
+    for (int d = threadIdx.x; d < hidden; d += blockDim.x) mean += to_f32(xr[d]);
+    mean = block_sum(mean, red) / (float)hidden;
+  }
   float ss = 0.f;
   for (int d = threadIdx.x; d < hidden; d += blockDim.x) {
-    const float v = to_f32(xr[d]);
+    const float v = to_f32(xr[d]) - mean;
     ss += v * v;
   }
   ss = block_sum(ss, red);
-  const float inv = rsqrtf(ss / (float)hidden + eps);
+  const float inv = kCenter ? 1.f / sqrtf(ss / (float)hidden + eps) : rsqrtf(ss / (float)hidden + eps);
   TO* o = out + (size_t)r * hidden;
   for (int d = threadIdx.x; d < hidden; d += blockDim.x)
-    o[d] = from_f32<TO>(to_f32(xr[d]) * inv * (w_offset + load_as_f32(w, w_dtype, d)));
+    o[d] = from_f32<TO>((to_f32(xr[d]) - mean) * inv * (w_offset + load_as_f32(w, w_dtype, d)));
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -94,13 +100,16 @@ __global__ void history_average_kernel(float* __restrict__ h, float* __restrict_
 // holds two copies per request, [slots][2][taps - 1][channels]: a step reads copy state_phase[request] and leaves the
 // state as it stands after the step in the other copy (the host turns the phase over when the step is committed), so
 // that rows which read the old state and rows which write the new one can run in one kernel.
+// in_bias / out_bias (float32 [channels] or null): added to every input (which then enters the state with it; what lies before
+// a sequence's start stays zero) and to the filter's result.
 // ---------------------------------------------------------------------------------------------
 template <typename TX, typename TO>
 __global__ void short_conv_kernel(TO* __restrict__ out, const TX* __restrict__ x, const void* __restrict__ w, int w_dtype,
                                   float* __restrict__ state, long long state_stride, const int* __restrict__ cu_seqlens,
                                   const int* __restrict__ token_req, const int* __restrict__ state_slots,
                                   const int* __restrict__ state_phase, int channels, int taps, int add_input,
-                                  long long x_stride, long long out_stride, int act, int tokens) {
+                                  long long x_stride, long long out_stride, int act, int tokens,
+                                  const float* __restrict__ in_bias, const float* __restrict__ out_bias) {
   pdl_start();
   if ((int)blockIdx.x >= tokens) {
     // behind the filter's blocks, one block per request (and chunk of channels) leaves the new state in the other copy:
@@ -114,7 +123,8 @@ __global__ void short_conv_kernel(TO* __restrict__ out, const TX* __restrict__ x
     for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < channels; c += gridDim.y * blockDim.x)
       for (int k = 0; k < keep; ++k) {
         const int s = n + k - keep;
-        st[(size_t)k * channels + c] = s >= 0 ? to_f32(x[(size_t)(start + s) * x_stride + c]) : old[(size_t)(k + n) * channels + c];
+        st[(size_t)k * channels + c] = s >= 0 ? to_f32(x[(size_t)(start + s) * x_stride + c]) + (in_bias ? in_bias[c] : 0.f)
+                                              : old[(size_t)(k + n) * channels + c];
       }
     return;
   }
@@ -126,13 +136,14 @@ __global__ void short_conv_kernel(TO* __restrict__ out, const TX* __restrict__ x
   const float* st = (req >= 0 && keep > 0) ? state + (size_t)state_slots[req] * state_stride + (size_t)state_phase[req] * keep * channels
                                            : nullptr;
   for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < channels; c += gridDim.y * blockDim.x) {
-    const float cur = to_f32(x[(size_t)t * x_stride + c]);
-    float acc = add_input ? cur : 0.f;
+    const float ib = in_bias ? in_bias[c] : 0.f;
+    const float cur = to_f32(x[(size_t)t * x_stride + c]) + ib;
+    float acc = (add_input ? cur : 0.f) + (out_bias ? out_bias[c] : 0.f);
     for (int j = 0; j < taps; ++j) {
       const int s = rel - keep + j;
       float v;
       if (s >= 0)
-        v = to_f32(x[(size_t)(start + s) * x_stride + c]);
+        v = to_f32(x[(size_t)(start + s) * x_stride + c]) + ib;
       else
         v = st ? st[(size_t)(keep + s) * channels + c] : 0.f;
       acc += load_as_f32(w, w_dtype, (size_t)c * taps + j) * v;
@@ -284,6 +295,151 @@ __global__ void branch_norm_add_vec_kernel(float* __restrict__ h, const TA* __re
   }
 }
 
+// v = a, or ca rms(a; wa) + cb rms(b; wb) of two results that were computed side by side (kPair, eps pair_eps);
+// v <- (v - mean v) / sqrt(var v + eps) * w (kCenter: a layer norm) or v / sqrt(mean v^2 + eps) * w, when w is given;
+// h += v (when h is given; low: the new h in bfloat16), out = v (when out is given).
+// VPT: groups of four numbers a thread keeps in registers; 0: any width, the numbers are formed again for every pass.
+struct JoinArgs {
+  float* h;
+  const float* a;
+  const float* b;
+  const float* wa;
+  const float* wb;
+  float ca, cb, pair_eps;
+  const float* w;
+  float eps;
+  float* out;
+  bf16* low;
+  int hidden;
+};
+
+template <int VPT, bool kPair, bool kCenter>
+__global__ void branch_join_kernel(const JoinArgs p) {
+  pdl_trigger();
+  __shared__ float red[32], red2[32];
+  const int hidden = p.hidden;
+  const size_t row = (size_t)blockIdx.x * hidden;
+  const float n = (float)hidden;
+  if (VPT > 0) {
+    constexpr int N = VPT > 0 ? VPT : 1;
+    const int nvec = hidden / 4;
+    float av[N][4], bv[N][4], wv[N][4], wb[N][4];
+#pragma unroll
+    for (int k = 0; k < N; ++k) {        // weights do not depend on the kernels ahead on the stream
+      const int v = threadIdx.x + k * blockDim.x;
+      if (v < nvec && kPair) {
+        load4(p.wa + (size_t)v * 4, wv[k]);
+        load4(p.wb + (size_t)v * 4, wb[k]);
+      }
+    }
+    pdl_wait();
+    float hv[N][4], nw[N][4];
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      const int v = threadIdx.x + k * blockDim.x;
+      const size_t at = row + (size_t)v * 4;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) av[k][e] = bv[k][e] = hv[k][e] = nw[k][e] = 0.f;
+      if (v < nvec) {
+        load4(p.a + at, av[k]);
+        if (kPair) load4(p.b + at, bv[k]);
+        if (p.h) load4(p.h + at, hv[k]);
+        if (p.w) load4(p.w + (size_t)v * 4, nw[k]);
+      }
+    }
+    if (kPair) {
+      float sa = 0.f, sb = 0.f;
+#pragma unroll
+      for (int k = 0; k < N; ++k)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sa += av[k][e] * av[k][e], sb += bv[k][e] * bv[k][e];
+      sa = block_sum(sa, red);
+      sb = block_sum(sb, red2);
+      const float ia = p.ca / sqrtf(sa / n + p.pair_eps), ib = p.cb / sqrtf(sb / n + p.pair_eps);
+#pragma unroll
+      for (int k = 0; k < N; ++k) {
+        const int v = threadIdx.x + k * blockDim.x;
+        if (v < nvec)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) av[k][e] = av[k][e] * ia * wv[k][e] + bv[k][e] * ib * wb[k][e];
+      }
+    }
+    if (p.w) {
+      float mean = 0.f;
+      if (kCenter) {
+#pragma unroll
+        for (int k = 0; k < N; ++k)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) mean += av[k][e];
+        mean = block_sum(mean, red) / n;
+      }
+      float ss = 0.f;
+#pragma unroll
+      for (int k = 0; k < N; ++k) {
+        if ((int)threadIdx.x + k * (int)blockDim.x < nvec)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            av[k][e] -= mean;
+            ss += av[k][e] * av[k][e];
+          }
+      }
+      ss = block_sum(ss, red2);
+      const float inv = 1.f / sqrtf(ss / n + p.eps);
+#pragma unroll
+      for (int k = 0; k < N; ++k)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) av[k][e] = av[k][e] * inv * nw[k][e];
+    }
+#pragma unroll
+    for (int k = 0; k < N; ++k) {
+      const int v = threadIdx.x + k * blockDim.x;
+      if (v >= nvec) continue;
+      const size_t at = row + (size_t)v * 4;
+      if (p.out) store4(p.out + at, av[k]);
+      if (p.h) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) hv[k][e] += av[k][e];
+        store4(p.h + at, hv[k]);
+        if (p.low) store4(p.low + at, hv[k]);
+      }
+    }
+    return;
+  }
+  pdl_wait();
+  float ia = 1.f, ib = 0.f;
+  if (kPair) {
+    float sa = 0.f, sb = 0.f;
+    for (int d = threadIdx.x; d < hidden; d += blockDim.x) sa += p.a[row + d] * p.a[row + d], sb += p.b[row + d] * p.b[row + d];
+    sa = block_sum(sa, red);
+    sb = block_sum(sb, red2);
+    ia = p.ca / sqrtf(sa / n + p.pair_eps), ib = p.cb / sqrtf(sb / n + p.pair_eps);
+  }
+  auto value = [&](int d) { return kPair ? p.a[row + d] * ia * p.wa[d] + p.b[row + d] * ib * p.wb[d] : p.a[row + d]; };
+  float mean = 0.f, inv = 1.f;
+  if (p.w) {
+    if (kCenter) {
+      for (int d = threadIdx.x; d < hidden; d += blockDim.x) mean += value(d);
+      mean = block_sum(mean, red) / n;
+    }
+    float ss = 0.f;
+    for (int d = threadIdx.x; d < hidden; d += blockDim.x) {
+      const float v = value(d) - mean;
+      ss += v * v;
+    }
+    ss = block_sum(ss, red2);
+    inv = 1.f / sqrtf(ss / n + p.eps);
+  }
+  for (int d = threadIdx.x; d < hidden; d += blockDim.x) {
+    const float v = p.w ? (value(d) - mean) * inv * p.w[d] : value(d);
+    if (p.out) p.out[row + d] = v;
+    if (p.h) {
+      const float next = p.h[row + d] + v;
+      p.h[row + d] = next;
+      if (p.low) p.low[row + d] = __float2bfloat16_rn(next);
+    }
+  }
+}
+
 // kConvRows consecutive rows and four channels per thread: a row's earlier inputs stay in registers while the thread
 // walks down its rows (rows of one request are consecutive), the taps' weights are read once, and only a request's
 // first rows of the step go to its state. The same launch leaves the new state: blocks behind the filter's own, one per
@@ -295,10 +451,19 @@ __global__ void __launch_bounds__(256) short_conv_vec_kernel(
     TO* __restrict__ out, const TX* __restrict__ x, const void* __restrict__ w, int w_dtype, float* __restrict__ state,
     long long state_stride, const int* __restrict__ cu_seqlens, const int* __restrict__ token_req,
     const int* __restrict__ state_slots, const int* __restrict__ state_phase, int tokens, int channels, int taps, int add_input,
-    int conv_blocks, long long x_stride, long long out_stride, int act) {
+    int conv_blocks, long long x_stride, long long out_stride, int act, const float* __restrict__ in_bias,
+    const float* __restrict__ out_bias) {
   pdl_trigger();
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
   const int keep = taps - 1;
+  float ib[4] = {0.f, 0.f, 0.f, 0.f}, ob[4] = {0.f, 0.f, 0.f, 0.f};
+  if (in_bias && c < channels) load4(in_bias + c, ib);
+  if (out_bias && c < channels) load4(out_bias + c, ob);
+  auto load_in = [&](const TX* p, float (&v)[4]) {
+    load4(p, v);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[e] += ib[e];
+  };
   if ((int)blockIdx.x >= conv_blocks) {
     // The blocks behind the filter's own: one per request, they leave the state as it stands after the step in the copy
     // that the step does not read (the filter's blocks read the other one, so the two kinds of block never meet).
@@ -312,7 +477,7 @@ __global__ void __launch_bounds__(256) short_conv_vec_kernel(
     for (int k = 0; k < keep; ++k) {
       const int s = n + k - keep;
       float v[4];
-      if (s >= 0) load4(x + (size_t)(start + s) * x_stride + c, v);
+      if (s >= 0) load_in(x + (size_t)(start + s) * x_stride + c, v);
       else load4(old + (size_t)(k + n) * channels + c, v);
       store4(nx + (size_t)k * channels + c, v);
     }
@@ -335,7 +500,7 @@ __global__ void __launch_bounds__(256) short_conv_vec_kernel(
 #pragma unroll
   for (int j = 0; j < kTaps; ++j) {
     const int r = t0 - 1 - j;
-    if (j < keep && r >= 0) load4(x + (size_t)r * x_stride + c, ring[j]);
+    if (j < keep && r >= 0) load_in(x + (size_t)r * x_stride + c, ring[j]);
   }
   const int t_end = min(tokens, t0 + kConvRows);
   // The requests of the rows and of the taps - 1 rows above them, and the rows' inputs: all asked for before any is used.
@@ -349,7 +514,7 @@ __global__ void __launch_bounds__(256) short_conv_vec_kernel(
   }
 #pragma unroll
   for (int i = 0; i < kConvRows; ++i)
-    if (t0 + i < t_end) load4(x + (size_t)(t0 + i) * x_stride + c, curs[i]);
+    if (t0 + i < t_end) load_in(x + (size_t)(t0 + i) * x_stride + c, curs[i]);
 #pragma unroll
   for (int i = 0; i < kConvRows; ++i) {
     const int t = t0 + i;
@@ -367,7 +532,7 @@ __global__ void __launch_bounds__(256) short_conv_vec_kernel(
     for (int e = 0; e < 4; ++e) cur[e] = curs[i][e];
     float acc[4];
 #pragma unroll
-    for (int e = 0; e < 4; ++e) acc[e] = add_input ? cur[e] : 0.f;
+    for (int e = 0; e < 4; ++e) acc[e] = (add_input ? cur[e] : 0.f) + ob[e];
 #pragma unroll
     for (int j = 0; j < kTaps; ++j) {     // j = 0: the row itself; j > 0: the input j rows above
       if (j >= taps) break;
@@ -450,14 +615,16 @@ int flat_blocks(long long n) {
 
 }  // namespace
 
-OI_API int oi_rmsnorm_cast(void* out, int out_dtype, const void* x, int x_dtype, const void* w, int w_dtype, const int* row_idx,
-                           int rows, int hidden, float eps, float w_offset, void* stream) {
-  OI_REQUIRE(rows >= 0 && hidden > 0, "rmsnorm_cast: bad sizes rows=%d hidden=%d", rows, hidden);
+namespace {
+template <bool kCenter>
+int norm_cast(void* out, int out_dtype, const void* x, int x_dtype, const void* w, int w_dtype, const int* row_idx, int rows,
+              int hidden, float eps, float w_offset, void* stream) {
+  OI_REQUIRE(rows >= 0 && hidden > 0, "norm_cast: bad sizes rows=%d hidden=%d", rows, hidden);
   if (rows == 0) return OI_OK;
   cudaStream_t s = (cudaStream_t)stream;
 #define OI_CAST_CASE(XD, OD, TX, TO)                                                                                  \
   if (x_dtype == XD && out_dtype == OD) {                                                                             \
-    oi_launch(rmsnorm_cast_kernel<TX, TO>, rows, kRowThreads, 0, s, (TO*)out, (const TX*)x, w, w_dtype, row_idx, hidden, eps, \
+    oi_launch(rmsnorm_cast_kernel<TX, TO, kCenter>, rows, kRowThreads, 0, s, (TO*)out, (const TX*)x, w, w_dtype, row_idx, hidden, eps, \
               w_offset);                                                                                              \
     OI_CHECK_LAUNCH();                                                                                                \
     return OI_OK;                                                                                                     \
@@ -467,7 +634,52 @@ OI_API int oi_rmsnorm_cast(void* out, int out_dtype, const void* x, int x_dtype,
   OI_CAST_CASE(OI_BF16, OI_F32, bf16, float)
   OI_CAST_CASE(OI_BF16, OI_BF16, bf16, bf16)
 #undef OI_CAST_CASE
-  OI_REQUIRE(false, "rmsnorm_cast: unknown dtype codes %d -> %d", x_dtype, out_dtype);
+  OI_REQUIRE(false, "norm_cast: unknown dtype codes %d -> %d", x_dtype, out_dtype);
+}
+}  // namespace
+
+OI_API int oi_rmsnorm_cast(void* out, int out_dtype, const void* x, int x_dtype, const void* w, int w_dtype, const int* row_idx,
+                           int rows, int hidden, float eps, float w_offset, void* stream) {
+  return norm_cast<false>(out, out_dtype, x, x_dtype, w, w_dtype, row_idx, rows, hidden, eps, w_offset, stream);
+}
+
+// the same with the row's mean taken off first (a layer norm without a bias)
+OI_API int oi_layernorm_cast(void* out, int out_dtype, const void* x, int x_dtype, const void* w, int w_dtype, const int* row_idx,
+                             int rows, int hidden, float eps, float w_offset, void* stream) {
+  return norm_cast<true>(out, out_dtype, x, x_dtype, w, w_dtype, row_idx, rows, hidden, eps, w_offset, stream);
+}
+
+// h (or null), a, b (or null), out (or null) float32 [rows, hidden]; wa, wb, w float32 [hidden] (w null: no norm of the result);
+// low bfloat16 [rows, hidden] or null. See branch_join_kernel.
+OI_API int oi_branch_join(float* h, const float* a, const float* b, const float* wa, const float* wb, float ca, float cb,
+                          float pair_eps, const float* w, int center, float eps, float* out, void* low, int rows, int hidden,
+                          void* stream) {
+  OI_REQUIRE(rows >= 0 && hidden > 0 && a != nullptr && (h != nullptr || out != nullptr), "branch_join: bad sizes rows=%d hidden=%d", rows, hidden);
+  OI_REQUIRE(b == nullptr || (wa != nullptr && wb != nullptr), "branch_join: two results need the weights of their norms");
+  if (rows == 0) return OI_OK;
+  cudaStream_t s = (cudaStream_t)stream;
+  const JoinArgs j{h, a, b, wa, wb, ca, cb, pair_eps, w, eps, out, (bf16*)low, hidden};
+  const int nvec = hidden / 4;
+  const bool vec = hidden % 4 == 0 && nvec <= 512 * 4 && aligned16(h) && aligned16(a) && aligned16(b) && aligned16(wa) && aligned16(wb) &&
+                   aligned16(w) && aligned16(out) && aligned16(low);
+#define OI_JOIN(V, PAIR, CENTER) oi_launch(branch_join_kernel<V, PAIR, CENTER>, rows, threads, 0, s, j)
+#define OI_JOIN_V(V)                                                                     \
+  do {                                                                                   \
+    if (b != nullptr) { if (center) OI_JOIN(V, true, true); else OI_JOIN(V, true, false); } \
+    else { if (center) OI_JOIN(V, false, true); else OI_JOIN(V, false, false); }         \
+  } while (0)
+  if (vec) {
+    const int vpt = nvec <= 256 ? 1 : (nvec <= 1024 ? 2 : 4);
+    const int threads = (((nvec + vpt - 1) / vpt + 31) / 32) * 32;
+    if (vpt == 1) OI_JOIN_V(1); else if (vpt == 2) OI_JOIN_V(2); else OI_JOIN_V(4);
+  } else {
+    const int threads = kRowThreads;
+    OI_JOIN_V(0);
+  }
+#undef OI_JOIN_V
+#undef OI_JOIN
+  OI_CHECK_LAUNCH();
+  return OI_OK;
 }
 
 OI_API int oi_branch_norm_add(float* h, const void* a, int a_dtype, const void* w, int w_dtype, int rows, int hidden, float eps,
@@ -518,11 +730,12 @@ OI_API int oi_history_average(float* h, float* hist, long long hist_stride, int 
 }
 
 // x_stride / out_stride: elements between rows (the channels of a row may be a slice of a wider buffer); act: OI_ACT_NONE
-// or OI_ACT_SILU on the filter's result. The state keeps the INPUTS, so the activation does not touch it.
+// or OI_ACT_SILU on the filter's result; in_bias / out_bias: see short_conv_kernel. The state keeps the INPUTS, so the activation does not touch it.
 OI_API int oi_short_conv_strided(void* out, int out_dtype, long long out_stride, const void* x, int x_dtype, long long x_stride,
                                  const void* w, int w_dtype, float* state, long long state_stride, const int* cu_seqlens,
                                  const int* token_req, const int* state_slots, const int* state_phase, int tokens, int requests,
-                                 int channels, int taps, int add_input, int update_state, int act, void* stream) {
+                                 int channels, int taps, int add_input, int update_state, int act, const float* in_bias,
+                                 const float* out_bias, void* stream) {
   OI_REQUIRE(act == OI_ACT_NONE || act == OI_ACT_SILU, "short_conv: unknown activation code %d", act);
   OI_REQUIRE(x_stride >= channels && out_stride >= channels, "short_conv: rows narrower than the channels");
   OI_REQUIRE(tokens >= 0 && requests >= 0 && channels > 0 && taps >= 1, "short_conv: bad sizes tokens=%d channels=%d taps=%d",
@@ -535,14 +748,15 @@ OI_API int oi_short_conv_strided(void* out, int out_dtype, long long out_stride,
   const dim3 grid(tokens, cy);
   const bool vec = x_stride % 4 == 0 && out_stride % 4 == 0 && channels % 4 == 0 && taps <= kConvMaxTaps && aligned16(out) &&
                    aligned16(x) &&
-                   (taps == 1 || (aligned16(state) && state_stride % 4 == 0));
+                   (taps == 1 || (aligned16(state) && state_stride % 4 == 0)) && aligned16(in_bias) && aligned16(out_bias);
   const int vthreads = channels / 4 >= 256 ? 256 : ((channels / 4 + 31) / 32) * 32;
   // the filter's blocks, and behind them one block per request (and chunk of channels) that leaves the new state
   const int conv_blocks = (tokens + kConvRows - 1) / kConvRows;
   const dim3 vgrid(conv_blocks + ((update_state && taps > 1) ? requests : 0), vec ? (channels / 4 + vthreads - 1) / vthreads : 1);
 #define OI_CONV_VEC(TX, TO, KT)                                                                                          \
   oi_launch(short_conv_vec_kernel<TX, TO, KT>, vgrid, vthreads, 0, s, (TO*)out, (const TX*)x, w, w_dtype, state, state_stride, \
-            cu_seqlens, token_req, state_slots, state_phase, tokens, channels, taps, add_input, conv_blocks, x_stride, out_stride, act)
+            cu_seqlens, token_req, state_slots, state_phase, tokens, channels, taps, add_input, conv_blocks, x_stride, out_stride, act, \
+            in_bias, out_bias)
 #define OI_CONV_CASE(XD, OD, TX, TO)                                                                                     \
   if (x_dtype == XD && out_dtype == OD) {                                                                                \
     if (vec) {                                                                                                           \
@@ -555,7 +769,7 @@ OI_API int oi_short_conv_strided(void* out, int out_dtype, long long out_stride,
     /* the filter's blocks, and behind them one block per request (and chunk of channels) that leaves the new state */    \
     oi_launch(short_conv_kernel<TX, TO>, dim3(tokens + ((update_state && taps > 1) ? requests : 0), cy), kRowThreads, 0, s, \
               (TO*)out, (const TX*)x, w, w_dtype, state, state_stride, cu_seqlens, token_req, state_slots, state_phase,  \
-              channels, taps, add_input, x_stride, out_stride, act, tokens);                                             \
+              channels, taps, add_input, x_stride, out_stride, act, tokens, in_bias, out_bias);                                             \
     OI_CHECK_LAUNCH();                                                                                                   \
     return OI_OK;                                                                                                        \
   }
@@ -572,7 +786,8 @@ OI_API int oi_short_conv(void* out, int out_dtype, const void* x, int x_dtype, c
                          const int* state_phase, int tokens, int requests, int channels, int taps, int add_input, int update_state,
                          void* stream) {
   return oi_short_conv_strided(out, out_dtype, channels, x, x_dtype, channels, w, w_dtype, state, state_stride, cu_seqlens, token_req,
-                               state_slots, state_phase, tokens, requests, channels, taps, add_input, update_state, OI_ACT_NONE, stream);
+                               state_slots, state_phase, tokens, requests, channels, taps, add_input, update_state, OI_ACT_NONE,
+                               nullptr, nullptr, stream);
 }
 
 OI_API int oi_latent_store(void* pages, long long page_stride, int page_size, int row_elems, const void* src, long long src_stride,

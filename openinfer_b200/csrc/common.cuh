@@ -203,4 +203,12 @@ __device__ __forceinline__ float block_max(float v, float* scratch) {
   return r;
 }
 
+// The first key that the query at position `pos` sees. window 0: every key; > 0: the last `window` keys, its own included;
+// < 0: the keys of its own chunk of -window positions (chunks are counted from a sequence's position 0). Never falls as pos rises.
+__host__ __device__ __forceinline__ int first_visible(int pos, int window) {
+  if (window > 0) return pos - window + 1 > 0 ? pos - window + 1 : 0;
+  if (window < 0) return pos - pos % -window;
+  return 0;
+}
+
 static inline int ceil_div(long long a, long long b) { return (int)((a + b - 1) / b); }

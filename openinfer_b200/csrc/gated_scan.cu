@@ -3,7 +3,10 @@
 //   z = sigmoid(zl + bz),  u = ul + bx,  c = u + 1/2 for u >= 0 and sigmoid(u) below,
 //   S_t = (1 - z_t) S_(t-1) + z_t c_t  (float32, zero at a request's start),  y_t = S_t * silu(g_t)
 //
-// zl, ul and g are columns of one fused product's float32 sums. A block owns a request and 32 channels and walks the request's
+// and, with coefficients formed elsewhere (csrc/block_gates.cu), the affine recurrence S_t = a_t S_(t-1) + b_t,
+// y_t = S_t * gelu_tanh(g_t + bg).
+//
+// zl, ul and g (or a, b and g) are columns of float32 buffers. A block owns a request and 32 channels and walks the request's
 // rows 256 at a time: a thread takes four channels of a run of four rows, forms the run's composition S -> A S + B, and after
 // an exchange inside the warp and one through shared memory starts from the state behind the runs in front of it. The sums
 // arrive by cp.async, two rounds deep. Only one block reads and writes a channel's state, so there is one copy of it. Requests
@@ -43,10 +46,18 @@ __device__ __forceinline__ void store4(bf16* o, const float (&v)[4]) {
   *reinterpret_cast<uint2*>(o) = t;
 }
 
-template <typename TO, bool kFast>
+// what the state is multiplied by on its way out
+template <bool kFast>
+__device__ __forceinline__ float gelu_tanh_f(float z) {
+  const float t = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+  return kFast ? div_f<true>(z, 1.f + exp_f<true>(-2.f * t)) : 0.5f * z * (1.f + tanhf(t));
+}
+
+// kAffine: col 0 and col_step of `zug` hold a and b themselves, and `bias` [channels] is that of the output gate
+template <typename TO, bool kFast, bool kAffine>
 __global__ void __launch_bounds__(kWarps * 32)
 mingru_scan_kernel(TO* __restrict__ out, long long out_stride, const float* __restrict__ zug, long long stride, int col_step,
-                   const float* __restrict__ bias, float* __restrict__ state, long long state_stride, const int* __restrict__ cu_seqlens,
+                   const float* __restrict__ gate, long long gate_stride, const float* __restrict__ bias, float* __restrict__ state, long long state_stride, const int* __restrict__ cu_seqlens,
                    const int* __restrict__ token_req, const int* __restrict__ state_slots, int channels, int whole_fours) {
   pdl_start();
   __shared__ float4 sa[2][kWarps][8], sb[2][kWarps][8];
@@ -62,12 +73,13 @@ mingru_scan_kernel(TO* __restrict__ out, long long out_stride, const float* __re
 #pragma unroll
   for (int k = 0; k < 4; ++k) {
     const bool in = cc + k < channels;
-    bz[k] = in ? bias[cc + k] : 0.f;
-    bx[k] = in ? bias[channels + cc + k] : 0.f;
+    bz[k] = in ? bias[cc + k] : 0.f;                 // (kAffine: the output gate's)
+    bx[k] = in && !kAffine ? bias[channels + cc + k] : 0.f;
     S[k] = in ? st[k] : 0.f;
   }
   constexpr int kWalk = kWarps * 4 * kRows;        // rows of a round
   const float* base = zug + (size_t)start * stride + cc;
+  const float* gate_base = gate + (size_t)start * gate_stride + cc;
   TO* o_base = out + (size_t)start * out_stride + cc;
   constexpr int kThreads = kWarps * 32;
   float4* const mine_in = stage + threadIdx.x;
@@ -75,11 +87,12 @@ mingru_scan_kernel(TO* __restrict__ out, long long out_stride, const float* __re
     if (t0 < n) {
 #pragma unroll
       for (int i = 0; i < kRows; ++i) {
-        const float* p = base + (size_t)min(t0 + (warp * 4 + run) * kRows + i, n - 1) * stride;
+        const int r = min(t0 + (warp * 4 + run) * kRows + i, n - 1);
+        const float* p = base + (size_t)r * stride;
 #pragma unroll
         for (int k = 0; k < 3; ++k) {
           const unsigned dst = (unsigned)__cvta_generic_to_shared(mine_in + (turn * kRows * 3 + i * 3 + k) * kThreads);
-          asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(dst), "l"(p + k * col_step) : "memory");
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(dst), "l"(k < 2 ? p + k * col_step : gate_base + (size_t)r * gate_stride) : "memory");
         }
       }
     }
@@ -102,7 +115,10 @@ mingru_scan_kernel(TO* __restrict__ out, long long out_stride, const float* __re
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
         a[i][k] = 1.f, v[i][k] = 0.f;              // rows behind the last one leave the state as it is
-        if (first + i < n) keep_and_add<kFast>(z4[k] + bz[k], u4[k] + bx[k], a[i][k], v[i][k]);
+        if (first + i < n) {
+          if (kAffine) a[i][k] = z4[k], v[i][k] = u4[k], g[i][k] += bz[k];
+          else keep_and_add<kFast>(z4[k] + bz[k], u4[k] + bx[k], a[i][k], v[i][k]);
+        }
         A[k] *= a[i][k];
         B[k] = a[i][k] * B[k] + v[i][k];
       }
@@ -145,7 +161,7 @@ mingru_scan_kernel(TO* __restrict__ out, long long out_stride, const float* __re
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
         mine[k] = a[i][k] * mine[k] + v[i][k];
-        y[k] = mine[k] * silu_f<kFast>(g[i][k]);
+        y[k] = mine[k] * (kAffine ? gelu_tanh_f<kFast>(g[i][k]) : silu_f<kFast>(g[i][k]));
       }
       if (first + i < n && c < channels) {
         TO* o = o_base + (size_t)(first + i) * out_stride;
@@ -209,9 +225,9 @@ OI_API int oi_mingru_scan(void* out, int out_dtype, long long out_stride, const 
 #define OI_GRU(TO, FAST)                                                                                                   \
   do {                                                                                                                     \
     if (longer) {                                                                                                          \
-      OI_CHECK_CUDA(cudaFuncSetAttribute(mingru_scan_kernel<TO, FAST>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
-      oi_launch(mingru_scan_kernel<TO, FAST>, dim3(requests, (channels + kChannels - 1) / kChannels), kWarps * 32, smem, s, (TO*)out, \
-                out_stride, zug, stride, col_step, bias, state, state_stride, cu_seqlens, token_req, state_slots, channels, fours); \
+      OI_CHECK_CUDA(cudaFuncSetAttribute(mingru_scan_kernel<TO, FAST, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+      oi_launch(mingru_scan_kernel<TO, FAST, false>, dim3(requests, (channels + kChannels - 1) / kChannels), kWarps * 32, smem, s, (TO*)out, \
+                out_stride, zug, stride, col_step, zug + 2 * (size_t)col_step, stride, bias, state, state_stride, cu_seqlens, token_req, state_slots, channels, fours); \
       OI_CHECK_LAUNCH();                                                                                                   \
     }                                                                                                                      \
     if (singles)                                                                                                           \
@@ -222,6 +238,38 @@ OI_API int oi_mingru_scan(void* out, int out_dtype, long long out_stride, const 
   else if (out_dtype == OI_BF16) OI_GRU(bf16, true);
   else OI_REQUIRE(false, "mingru_scan: unknown dtype code %d", out_dtype);
 #undef OI_GRU
+  OI_CHECK_LAUNCH();
+  return OI_OK;
+}
+
+// ab float32 [tokens, ab_stride]: a at column 0, b at col_step; y float32 [tokens, y_stride] and y_bias [channels]: the output gate;
+// state float32 [slots, state_stride]; out [tokens, channels]. Requests that bring one row are left alone (oi_rglru_gates).
+OI_API int oi_affine_scan(void* out, int out_dtype, long long out_stride, const float* ab, long long ab_stride, int col_step,
+                          const float* y, long long y_stride, const float* y_bias, float* state, long long state_stride,
+                          const int* cu_seqlens, const int* token_req, const int* state_slots, int tokens, int requests, int channels,
+                          void* stream) {
+  OI_REQUIRE(tokens >= 0 && requests >= 0 && channels > 0 && col_step >= channels && ab_stride >= (long long)col_step + channels &&
+             y_stride >= channels && out_stride >= channels && state_stride >= channels, "affine_scan: bad sizes tokens=%d channels=%d", tokens, channels);
+  OI_REQUIRE(ab && y && y_bias && state && cu_seqlens && token_req && state_slots && out, "affine_scan: a buffer is missing");
+  if (tokens == 0 || requests == 0) return OI_OK;
+  // (the last four channels are read whole: the buffers' columns are padded to fours)
+  OI_REQUIRE(ab_stride % 4 == 0 && col_step % 4 == 0 && y_stride % 4 == 0 && ((uintptr_t)ab & 15) == 0 && ((uintptr_t)y & 15) == 0 &&
+             ab_stride >= (long long)col_step + ((channels + 3) & ~3) && y_stride >= ((channels + 3) & ~3),
+             "affine_scan: the coefficients must be readable 16 bytes at a time");
+  const int fours = channels % 4 == 0 && out_stride % 4 == 0 && ((uintptr_t)out & 15) == 0 ? 1 : 0;
+  cudaStream_t s = (cudaStream_t)stream;
+  const size_t smem = (size_t)2 * kRows * 3 * kWarps * 32 * sizeof(float4);
+  const dim3 grid(requests, (channels + kChannels - 1) / kChannels);
+#define OI_AFFINE(TO, FAST)                                                                                                       \
+  do {                                                                                                                            \
+    OI_CHECK_CUDA(cudaFuncSetAttribute(mingru_scan_kernel<TO, FAST, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+    oi_launch(mingru_scan_kernel<TO, FAST, true>, grid, kWarps * 32, smem, s, (TO*)out, out_stride, ab, ab_stride, col_step, y,    \
+              y_stride, y_bias, state, state_stride, cu_seqlens, token_req, state_slots, channels, fours);                         \
+  } while (0)
+  if (out_dtype == OI_F32) OI_AFFINE(float, false);
+  else if (out_dtype == OI_BF16) OI_AFFINE(bf16, true);
+  else OI_REQUIRE(false, "affine_scan: unknown dtype code %d", out_dtype);
+#undef OI_AFFINE
   OI_CHECK_LAUNCH();
   return OI_OK;
 }

@@ -4,7 +4,11 @@
 //                          their softmax -> ids [rows, top], weights [rows, top]. Scoring 1 ("sigmoid, corrected, by groups"):
 //                          s = sigmoid(z); the choice goes by s + correction, among the experts of the `keep_groups` best of
 //                          `n_groups` equal groups of neighbours (a group's score: the sum of its two largest choice scores);
-//                          the weights are the chosen experts' s divided by their sum (+ 1e-20)
+//                          the weights are the chosen experts' s divided by their sum (+ 1e-20). Scoring 2 ("softmax, corrected,
+//                          by groups"): s = softmax(z) over all rows of the router; a group's score: its largest choice score;
+//                          the weights are the chosen s times weight_scale. The router may have more rows than there are
+//                          experts: a choice behind the last expert stands for the row itself (it has no weights; the row
+//                          times the choice's weight is added in step 4)
 //   2. moe_group_kernel    the (row, choice) pairs sorted by expert (stable, so the order never depends on timing), and
 //                          the list of row tiles (expert, first sorted place, rows) the products run over
 //   3. moe_gemm_kernel     per tile: act(x W_gate_e^T, x W_up_e^T) for the rows of the tile, gathered by their pair's row;
@@ -27,7 +31,7 @@ constexpr int kMaxTop = 32;
 template <typename T>
 __global__ void moe_router_kernel(const T* __restrict__ x, long long ldx, const void* __restrict__ w, int w_dtype, int rows, int K,
                                   int E, int top, int* __restrict__ ids, float* __restrict__ wts, int scoring,
-                                  const float* __restrict__ correction, int n_groups, int keep_groups) {
+                                  const float* __restrict__ correction, int n_groups, int keep_groups, float weight_scale) {
   pdl_start();
   extern __shared__ float smem[];              // the row's logits [E], scores [E], group scores [E], then which are taken [E bytes]
   const int warps = blockDim.x >> 5, wi = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -81,11 +85,18 @@ __global__ void moe_router_kernel(const T* __restrict__ x, long long ldx, const 
   }
   __syncthreads();
   if (wi != 0) return;
-  if (scoring == 1) {
+  if (scoring != 0) {
+    float top_z = -INFINITY, sum = 0.f;
+    if (scoring == 2) {                              // softmax over all of them
+      for (int e = lane; e < E; e += 32) top_z = fmaxf(top_z, z[e]);
+      top_z = warp_max(top_z);
+      for (int e = lane; e < E; e += 32) sum += expf(z[e] - top_z);
+      sum = warp_sum(sum);
+    }
     for (int e = lane; e < E; e += 32) {
-      const float sg = 1.f / (1.f + expf(-z[e]));
-      sc[e] = sg;
-      z[e] = sg + (correction ? correction[e] : 0.f);
+      const float s = scoring == 2 ? expf(z[e] - top_z) / sum : 1.f / (1.f + expf(-z[e]));
+      sc[e] = s;
+      z[e] = s + (correction ? correction[e] : 0.f);
     }
     __syncwarp();
     if (n_groups > 1 && keep_groups < n_groups) {
@@ -96,7 +107,7 @@ __global__ void moe_router_kernel(const T* __restrict__ x, long long ldx, const 
           const float v = z[g * per + i];
           if (v > a) { b = a; a = v; } else if (v > b) { b = v; }
         }
-        gs[g] = per > 1 ? a + b : a;
+        gs[g] = scoring == 1 && per > 1 ? a + b : a;
       }
       __syncwarp();
       for (int e = lane; e < E; e += 32) taken[e] = 1;
@@ -150,7 +161,12 @@ __global__ void moe_router_kernel(const T* __restrict__ x, long long ldx, const 
     chosen_z[j] = best;
     chosen_e[j] = be;
   }
-  if (lane == 0 && scoring == 1) {
+  if (lane == 0 && scoring == 2) {
+    for (int j = 0; j < top; ++j) {
+      ids[(size_t)row * top + j] = chosen_e[j];
+      wts[(size_t)row * top + j] = sc[chosen_e[j]] * weight_scale;
+    }
+  } else if (lane == 0 && scoring == 1) {
     float sum = 0.f;
     for (int j = 0; j < top; ++j) sum += sc[chosen_e[j]];
     for (int j = 0; j < top; ++j) {
@@ -558,10 +574,11 @@ __global__ void __launch_bounds__(256) moe_gemm_mma_big_kernel(const bf16* __res
 template <typename T, typename TO, bool kGlu>
 __global__ void __launch_bounds__(128) moe_gemv_kernel(const T* __restrict__ A, long long lda, int a_div, const T* __restrict__ Wt,
                                                        long long w_expert_stride, TO* __restrict__ out, long long ld_out,
-                                                       const int* __restrict__ ids, int N, int K, float limit, int act) {
+                                                       const int* __restrict__ ids, int E, int N, int K, float limit, int act) {
   pdl_wait();    // no early trigger: waiting blocks of the next kernel would share the SMs with this product
   extern __shared__ __align__(16) float xs[];
   constexpr int kVec = 16 / (int)sizeof(T), kRows = 16;
+  if (ids[blockIdx.x] >= E) return;      // a choice that stands for the row itself
   const int p = blockIdx.x, lane = threadIdx.x & 31, wi = threadIdx.x >> 5;
   const T* xr = A + (size_t)(a_div > 0 ? p / a_div : p) * lda;
   for (int k = threadIdx.x; k < K; k += blockDim.x) xs[k] = to_f32(xr[k]);
@@ -622,16 +639,66 @@ __global__ void __launch_bounds__(128) moe_gemv_kernel(const T* __restrict__ A, 
   }
 }
 
-// add (or null): a float32 term per output number that every row gets beside its experts' sum (an expert all rows share)
+// add (or null): a float32 term per output number that every row gets beside its experts' sum (an expert all rows share);
+// x: the rows themselves, for choices behind the last of the E experts
+template <typename T>
 __global__ void moe_combine_kernel(float* __restrict__ out, const float* __restrict__ y, const float* __restrict__ wts, int top, int W,
-                                   size_t n, const float* __restrict__ add) {
+                                   size_t n, const float* __restrict__ add, const int* __restrict__ ids, int E, const T* __restrict__ x,
+                                   long long ldx) {
   pdl_start();
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
     const size_t t = i / W, c = i - t * W;
     float acc = 0.f;
-    for (int j = 0; j < top; ++j) acc += wts[t * top + j] * y[(t * top + j) * W + c];
+    for (int j = 0; j < top; ++j)
+      acc += wts[t * top + j] * (ids[t * top + j] < E ? y[(t * top + j) * W + c] : to_f32(x[t * (size_t)ldx + c]));
     out[i] = add ? acc + add[i] : acc;
   }
+}
+// four neighbouring numbers of a row a thread, 16 bytes of every expert's result at a time
+template <typename T>
+__global__ void moe_combine_vec_kernel(float* __restrict__ out, const float* __restrict__ y, const float* __restrict__ wts, int top, int W,
+                                       size_t n4, const float* __restrict__ add, const int* __restrict__ ids, int E,
+                                       const T* __restrict__ x, long long ldx) {
+  pdl_start();
+  const int w4 = W / 4;
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n4; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t t = i / w4, c = (i - t * w4) * 4;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int j = 0; j < top; ++j) {
+      const float w = wts[t * top + j];
+      float4 v;
+      if (ids[t * top + j] < E) {
+        v = *reinterpret_cast<const float4*>(y + (t * top + j) * W + c);
+      } else {
+        const T* r = x + t * (size_t)ldx + c;
+        v = make_float4(to_f32(r[0]), to_f32(r[1]), to_f32(r[2]), to_f32(r[3]));
+      }
+      acc.x += w * v.x, acc.y += w * v.y, acc.z += w * v.z, acc.w += w * v.w;
+    }
+    if (add) {
+      const float4 v = *reinterpret_cast<const float4*>(add + i * 4);
+      acc.x += v.x, acc.y += v.y, acc.z += v.z, acc.w += v.w;
+    }
+    *reinterpret_cast<float4*>(out + i * 4) = acc;
+  }
+}
+
+// the weighted sum of a row's choices, by the kernel that takes the width
+int launch_combine(float* out, const float* y, const float* wts, int top, int W, int rows, const float* add, const int* ids, int E,
+                   const void* x, int dtype, long long ldx, cudaStream_t s) {
+  const size_t n = (size_t)rows * W;
+  const bool vec = W % 4 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)y % 16 == 0 && (uintptr_t)add % 16 == 0;
+  const size_t work = vec ? n / 4 : n;
+  const int blocks = (int)((work + 255) / 256 > 148 * 16 ? 148 * 16 : (work + 255) / 256);
+#define OI_COMBINE(T)                                                                                                            \
+  do {                                                                                                                           \
+    if (vec) oi_launch(moe_combine_vec_kernel<T>, blocks, 256, 0, s, out, y, wts, top, W, work, add, ids, E, (const T*)x, ldx);  \
+    else oi_launch(moe_combine_kernel<T>, blocks, 256, 0, s, out, y, wts, top, W, work, add, ids, E, (const T*)x, ldx);          \
+  } while (0)
+  if (dtype == OI_F32) OI_COMBINE(float); else OI_COMBINE(bf16);
+#undef OI_COMBINE
+  OI_CHECK_LAUNCH();
+  return OI_OK;
 }
 
 }  // namespace
@@ -648,35 +715,37 @@ OI_API int oi_moe_small(int pairs, int experts) { return pairs <= 2 * experts &&
 // x [rows, K] (row stride ldx) in `dtype`; router weights [E, K]; ids, wts [rows, top]; sorted [rows * top];
 // tile_info [3 * max_tiles + 1] with max_tiles = oi_moe_max_tiles(rows * top, E).
 OI_API int oi_moe_route_scored(const void* x, int dtype, long long ldx, const void* w_router, int w_dtype, int rows, int K, int E,
-                               int top, int scoring, const float* correction, int n_groups, int keep_groups, int* ids, float* wts,
-                               int* sorted, int* tile_info, void* stream);
+                               int identity, int top, int scoring, const float* correction, int n_groups, int keep_groups,
+                               float weight_scale, int* ids, float* wts, int* sorted, int* tile_info, void* stream);
 
 OI_API int oi_moe_route(const void* x, int dtype, long long ldx, const void* w_router, int w_dtype, int rows, int K, int E, int top,
                         int* ids, float* wts, int* sorted, int* tile_info, void* stream) {
-  return oi_moe_route_scored(x, dtype, ldx, w_router, w_dtype, rows, K, E, top, 0, nullptr, 1, 1, ids, wts, sorted, tile_info, stream);
+  return oi_moe_route_scored(x, dtype, ldx, w_router, w_dtype, rows, K, E, 0, top, 0, nullptr, 1, 1, 1.f, ids, wts, sorted, tile_info, stream);
 }
 
 // scoring 0: the `top` largest logits, weighted by their softmax. scoring 1: sigmoid scores; the choice goes by score +
 // correction (float32 [E] or null) among the experts of the `keep_groups` best of `n_groups` equal groups of neighbours;
-// weights: the chosen scores (without the correction) divided by their sum.
+// weights: the chosen scores (without the correction) divided by their sum. scoring 2: softmax scores, see the file's head.
+// The router has E + identity rows, as have the correction and the groups together.
 OI_API int oi_moe_route_scored(const void* x, int dtype, long long ldx, const void* w_router, int w_dtype, int rows, int K, int E,
-                               int top, int scoring, const float* correction, int n_groups, int keep_groups, int* ids, float* wts,
-                               int* sorted, int* tile_info, void* stream) {
-  OI_REQUIRE(rows >= 0 && K > 0 && E > 0 && top > 0 && top <= E && top <= kMaxTop, "moe_route: bad sizes experts=%d top=%d (at most %d)", E,
-             top, kMaxTop);
-  OI_REQUIRE(E <= 4096, "moe_route: %d experts, at most 4096", E);
-  OI_REQUIRE(scoring == 0 || scoring == 1, "moe_route: unknown scoring %d", scoring);
-  OI_REQUIRE(n_groups >= 1 && keep_groups >= 1 && keep_groups <= n_groups && E % n_groups == 0 && (E / n_groups) * keep_groups >= top,
-             "moe_route: %d experts in %d groups of which %d are kept cannot give %d choices", E, n_groups, keep_groups, top);
+                               int identity, int top, int scoring, const float* correction, int n_groups, int keep_groups,
+                               float weight_scale, int* ids, float* wts, int* sorted, int* tile_info, void* stream) {
+  const int all = E + identity;
+  OI_REQUIRE(rows >= 0 && K > 0 && E > 0 && identity >= 0 && top > 0 && top <= all && top <= kMaxTop,
+             "moe_route: bad sizes experts=%d+%d top=%d (at most %d)", E, identity, top, kMaxTop);
+  OI_REQUIRE(all <= 3584, "moe_route: %d experts, at most 3584", all);      // the row's scores lie in shared memory
+  OI_REQUIRE(scoring >= 0 && scoring <= 2, "moe_route: unknown scoring %d", scoring);
+  OI_REQUIRE(n_groups >= 1 && keep_groups >= 1 && keep_groups <= n_groups && all % n_groups == 0 && (all / n_groups) * keep_groups >= top,
+             "moe_route: %d experts in %d groups of which %d are kept cannot give %d choices", all, n_groups, keep_groups, top);
   if (rows == 0) return OI_OK;
   cudaStream_t s = (cudaStream_t)stream;
-  const size_t smem = 3 * (size_t)E * sizeof(float) + (size_t)E + 16;
+  const size_t smem = 3 * (size_t)all * sizeof(float) + (size_t)all + 16;
   if (dtype == OI_F32)
-    oi_launch(moe_router_kernel<float>, rows, 128, smem, s, (const float*)x, ldx, w_router, w_dtype, rows, K, E, top, ids, wts, scoring,
-              correction, n_groups, keep_groups);
+    oi_launch(moe_router_kernel<float>, rows, 128, smem, s, (const float*)x, ldx, w_router, w_dtype, rows, K, all, top, ids, wts, scoring,
+              correction, n_groups, keep_groups, weight_scale);
   else if (dtype == OI_BF16)
-    oi_launch(moe_router_kernel<bf16>, rows, 128, smem, s, (const bf16*)x, ldx, w_router, w_dtype, rows, K, E, top, ids, wts, scoring,
-              correction, n_groups, keep_groups);
+    oi_launch(moe_router_kernel<bf16>, rows, 128, smem, s, (const bf16*)x, ldx, w_router, w_dtype, rows, K, all, top, ids, wts, scoring,
+              correction, n_groups, keep_groups, weight_scale);
   else
     OI_REQUIRE(false, "moe_route: unknown dtype code %d", dtype);
   OI_CHECK_LAUNCH();
@@ -730,29 +799,25 @@ OI_API int oi_moe_experts(const void* x, int dtype, long long ldx, const void* w
   if (rows == 0) return OI_OK;
   cudaStream_t s = (cudaStream_t)stream;
   const int pairs = rows * top, max_tiles = oi_moe_max_tiles(pairs, E);
-  const size_t n_out = (size_t)rows * W;
-  const int cblocks = (int)((n_out + 255) / 256 > 148 * 16 ? 148 * 16 : (n_out + 255) / 256);
   if (oi_moe_small(pairs, E) && (size_t)(W > F ? W : F) * sizeof(float) <= 48 * 1024) {
     const dim3 v1(pairs, (F + 15) / 16), v2(pairs, (W + 15) / 16);
     if (dtype == OI_F32) {
       oi_launch(moe_gemv_kernel<float, float, true>, v1, 128, (size_t)W * 4, s, (const float*)x, ldx, top, (const float*)w_gate_up,
-                (long long)2 * F * W, (float*)act, (long long)F, ids, F, W, limit, glu);
+                (long long)2 * F * W, (float*)act, (long long)F, ids, E, F, W, limit, glu);
       OI_CHECK_LAUNCH();
       oi_launch(moe_gemv_kernel<float, float, false>, v2, 128, (size_t)F * 4, s, (const float*)act, (long long)F, 0, (const float*)w_down,
-                (long long)W * F, y, (long long)W, ids, W, F, 0.f, 0);
+                (long long)W * F, y, (long long)W, ids, E, W, F, 0.f, 0);
     } else if (dtype == OI_BF16) {
       oi_launch(moe_gemv_kernel<bf16, bf16, true>, v1, 128, (size_t)W * 4, s, (const bf16*)x, ldx, top, (const bf16*)w_gate_up,
-                (long long)2 * F * W, (bf16*)act, (long long)F, ids, F, W, limit, glu);
+                (long long)2 * F * W, (bf16*)act, (long long)F, ids, E, F, W, limit, glu);
       OI_CHECK_LAUNCH();
       oi_launch(moe_gemv_kernel<bf16, float, false>, v2, 128, (size_t)F * 4, s, (const bf16*)act, (long long)F, 0, (const bf16*)w_down,
-                (long long)W * F, y, (long long)W, ids, W, F, 0.f, 0);
+                (long long)W * F, y, (long long)W, ids, E, W, F, 0.f, 0);
     } else {
       OI_REQUIRE(false, "moe_experts: unknown dtype code %d", dtype);
     }
     OI_CHECK_LAUNCH();
-    oi_launch(moe_combine_kernel, cblocks, 256, 0, s, out, (const float*)y, wts, top, W, n_out, add);
-    OI_CHECK_LAUNCH();
-    return OI_OK;
+    return launch_combine(out, y, wts, top, W, rows, add, ids, E, x, dtype, ldx, s);
   }
   const int tile_rows = oi_moe_tile_rows(pairs, E), subs = tile_rows / kTileM;
   const bool big = tile_rows == kBigM;
@@ -791,9 +856,5 @@ OI_API int oi_moe_experts(const void* x, int dtype, long long ldx, const void* w
     OI_REQUIRE(false, "moe_experts: unknown dtype code %d", dtype);
   }
   OI_CHECK_LAUNCH();
-  const size_t n = (size_t)rows * W;
-  const int blocks = (int)((n + 255) / 256 > 148 * 16 ? 148 * 16 : (n + 255) / 256);
-  oi_launch(moe_combine_kernel, blocks, 256, 0, s, out, (const float*)y, wts, top, W, n, add);
-  OI_CHECK_LAUNCH();
-  return OI_OK;
+  return launch_combine(out, y, wts, top, W, rows, add, ids, E, x, dtype, ldx, s);
 }

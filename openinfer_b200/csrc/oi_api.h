@@ -131,15 +131,20 @@ OI_API int oi_short_conv(void* out, int out_dtype, const void* x, int x_dtype, c
 OI_API int oi_short_conv_strided(void* out, int out_dtype, long long out_stride, const void* x, int x_dtype, long long
        x_stride, const void* w, int w_dtype, float* state, long long state_stride, const int* cu_seqlens, const int*
        token_req, const int* state_slots, const int* state_phase, int tokens, int requests, int channels, int taps, int
-       add_input, int update_state, int act, void* stream);
+       add_input, int update_state, int act, const float* in_bias, const float* out_bias, void* stream);
+OI_API int oi_layernorm_cast(void* out, int out_dtype, const void* x, int x_dtype, const void* w, int w_dtype, const int*
+       row_idx, int rows, int hidden, float eps, float w_offset, void* stream);
+OI_API int oi_branch_join(float* h, const float* a, const float* b, const float* wa, const float* wb, float ca, float cb, float
+       pair_eps, const float* w, int center, float eps, float* out, void* low, int rows, int hidden, void* stream);
 
 // elementwise.cu: every gated activation, the ones with a limit included (OI_ACT_SWIGLU_CLAMP)
 OI_API int oi_glu_act(void* out, const void* gate_up, int dtype, int rows, int inter, int block, int act, float limit,
        void* stream);
 
 // recurrent.cu: mixers with a matrix memory per head (mode 0: the mLSTM cell, 1: the gated delta rule, 2: linear attention
-// with one fixed decay per head, p0 = the decays [H]; q, k and v get their silu there, v in place in `qkv`)
-OI_API int oi_recurrent_record(int D);
+// with one fixed decay per head, p0 = the decays [H]; q, k and v get their silu there, v in place in `qkv`; 3: the gated delta
+// rule with one decay per head, whose logits are read from `gates` at f_off, p0 = dt [H], p1 = A [H])
+OI_API int oi_recurrent_record(int mode, int D);
 OI_API int oi_recurrent_scan(int mode, const float* qkv, long long ld_qkv, int q_off, int k_off, int v_off, const float*
        gates, long long ld_gates, int i_off, int f_off, const float* decay, long long ld_decay, const void* p0, const
        void* p1, int p_dtype, float cap, float q_scale, float* prep, float* state, long long state_stride, const int*
@@ -147,7 +152,7 @@ OI_API int oi_recurrent_scan(int mode, const float* qkv, long long ld_qkv, int q
        int tokens, int requests, int H, int G, int D, int V, void* stream);
 OI_API int oi_head_norm_gate(void* out, int out_dtype, long long ld_out, const float* o, long long ld_o, const float*
        gate, long long ld_gate, const void* w, int w_dtype, int w_stride, int tokens, int H, int V, float eps, float
-       scale, void* stream);
+       scale, int gate_act, void* stream);
 
 // sandwich_ops.cu: a Dynamic Tanh norm, dyt(v) = tanh(alpha v) w + b, between two sublayers of a float32 stream
 // (h += dyt(branch; post); out = dyt(h; pre), either half optional; row_idx: out is read from these rows of h), and the
@@ -181,7 +186,22 @@ OI_API int oi_sigmoid_attention_mma(const void* q, long long q_stride, void* out
 OI_API int oi_slice_sum_gate(const float* part, const int* row_splits, const int* row_base, void* out, int dtype, long long
        out_stride, const void* gate, long long gate_stride, int tokens, int cols, void* stream);
 
-// gated_scan.cu: a gated recurrence per channel, S <- (1 - z) S + z c(u)
+// joint_norm.cu: q | k | v rows: bias, a norm over all heads together, rotation of the pairs (d, d + half), cache write
+OI_API int oi_joint_norm_half_store(void* qkv, int dtype, long long row_stride, int tokens, int nq, int nkv, int hd, int qk_dim,
+       const float* bias, const float* q_w, const float* k_w, float eps, const float* cos_tab, const float* sin_tab, int rot_half,
+       int max_pos, const int* positions, const int* slots, void* k_cache, void* v_cache, long long page_stride, int page_size,
+       void* stream);
+
+// block_gates.cu: the gates of a real-gated linear recurrent unit (block-diagonal products), its coefficients, and its single rows
+OI_API int oi_rglru_gates(const float* u, long long ld_u, const void* w, int w_dtype, const float* bias, const float* rate, float*
+       ab, long long ld_ab, int col_step, const float* y, long long ld_y, const float* y_bias, void* out, int out_dtype, long long
+       ld_out, float* state, long long state_stride, const int* cu_seqlens, const int* token_req, const int* state_slots, int tokens,
+       int blocks, int size, void* stream);
+
+// gated_scan.cu: recurrences per channel: S <- (1 - z) S + z c(u), and S <- a S + b with given a and b
+OI_API int oi_affine_scan(void* out, int out_dtype, long long out_stride, const float* ab, long long ab_stride, int col_step,
+       const float* y, long long y_stride, const float* y_bias, float* state, long long state_stride, const int* cu_seqlens, const
+       int* token_req, const int* state_slots, int tokens, int requests, int channels, void* stream);
 OI_API int oi_mingru_scan(void* out, int out_dtype, long long out_stride, const float* zug, long long stride, int col_step, const
        float* bias, float* state, long long state_stride, const int* cu_seqlens, const int* token_req, const int* state_slots,
        int tokens, int requests, int channels, int singles, int longer, void* stream);
@@ -207,9 +227,12 @@ OI_API int oi_moe_experts(const void* x, int dtype, long long ldx, const void* w
 // scoring 1: sigmoid scores; the choice goes by score + correction (float32 [E] or null) among the experts of the
 // `keep_groups` best of `n_groups` equal groups of neighbours (a group's score: the sum of its two largest choice scores);
 // the weights are the chosen experts' scores, without the correction, divided by their sum.
+// scoring 2: softmax scores; the choice goes by score + correction among the `keep_groups` best groups (a group's score: its
+// largest choice score); the weights are the chosen scores times `weight_scale`.
+// The router has E + identity rows; the choices E .. E + identity - 1 stand for the row itself (the groups hold them too).
 OI_API int oi_moe_route_scored(const void* x, int dtype, long long ldx, const void* w_router, int w_dtype, int rows, int K, int E,
-                               int top, int scoring, const float* correction, int n_groups, int keep_groups, int* ids, float* wts,
-                               int* sorted, int* tile_info, void* stream);
+                               int identity, int top, int scoring, const float* correction, int n_groups, int keep_groups, float
+                               weight_scale, int* ids, float* wts, int* sorted, int* tile_info, void* stream);
 OI_API int oi_moe_route_table(const int* token_ids, const int* table, int rows, int vocab, int E, int top, int* ids, float*
        wts, int* sorted, int* tile_info, void* stream);
 
@@ -382,7 +405,7 @@ typedef struct OiAttnLayer {
   const float* cos_tab;      // [max_pos, rot_half] or null
   const float* sin_tab;
   int q_row_stride, out_row_stride, dtype;
-  int nq, nkv, hd, window;   // window 0: every key
+  int nq, nkv, hd, window;   // window 0: every key; > 0: the last `window` keys; < 0: the keys of the query's chunk of -window positions
   float scale, eps, w_offset;
   int norm_dtype, rot_half, max_pos;
   int interleaved;           // the rotation turns neighbours (2 d, 2 d + 1) instead of (d, d + half)

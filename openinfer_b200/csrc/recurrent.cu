@@ -8,6 +8,7 @@
 //   kGatedDelta (gated delta rule):  C <- diag(g) C;  d = beta (v - C^T k);  C <- C + k d^T;  o = C^T q, with k and q made
 //                                    unit vectors (1e-6 inside the root), q times q_scale, beta = sigmoid(zb) and one decay
 //                                    per key channel g = exp(-exp(A_h) softplus(a + dt))
+//   kDeltaHeadDecay:                 the gated delta rule with one decay per head, g = exp(-exp(A_h) softplus(a_h + dt_h))
 //   kLinearDecay (linear attention with one fixed decay per head, "lightning attention"):
 //                                    C <- lambda_h C + k v^T;  o = C^T q, with q, k and v through silu first and no other scale
 //
@@ -22,7 +23,7 @@
 
 namespace {
 
-enum : int { kMatrixMemory = 0, kGatedDelta = 1, kLinearDecay = 2 };
+enum : int { kMatrixMemory = 0, kGatedDelta = 1, kLinearDecay = 2, kDeltaHeadDecay = 3 };
 constexpr int kThreads = 128;
 constexpr int kMaxRegs = 16;   // key channels a thread holds of its column
 
@@ -30,12 +31,13 @@ struct ScanArgs {
   const float* qkv;            // [tokens, ld_qkv]: queries, keys (kv head major, D each) and values (head major, V each)
   long long ld_qkv;
   int q_off, k_off, v_off;
-  const float* gates;          // [tokens, ld_gates]: matrix memory: zi at i_off + h, zf at f_off + h; delta: zb at i_off + h
+  const float* gates;          // [tokens, ld_gates]: matrix memory: zi at i_off + h, zf at f_off + h; delta: zb at i_off + h;
+                               // delta with a decay per head: also a at f_off + h
   long long ld_gates;
   int i_off, f_off;
   const float* decay;          // delta: a [tokens, ld_decay], head major, D each
   long long ld_decay;
-  const void* p0;              // matrix memory: bias of zi [H]; delta: dt [H * D]; linear decay: lambda [H]
+  const void* p0;              // matrix memory: bias of zi [H]; delta: dt [H * D] (a decay per head: [H]); linear decay: lambda [H]
   const void* p1;              // matrix memory: bias of zf [H]; delta: A [H]
   int p_dtype;
   float cap, q_scale;
@@ -52,6 +54,11 @@ struct ScanArgs {
   int tokens, H, G, D, V;
 };
 
+// what a read-out is multiplied by for a gate's raw value z: sigmoid(z), or z sigmoid(z)
+__device__ __forceinline__ float gate_value(float z, int act) {
+  const float s = 1.f / (1.f + expf(-z));
+  return act == OI_ACT_SILU ? z * s : s;
+}
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
 // Everything of a row that does not depend on the rows before it, one warp per (row, head), so that the scan's loop is
@@ -106,6 +113,71 @@ __global__ void recurrent_prepare_kernel(ScanArgs a) {
       rec[2 * D + d] = expf(-rate * softplus_f(x));
     }
     if (lane == 0) rec[3 * D] = 1.f / (1.f + expf(-gr[a.i_off + h]));
+  }
+}
+
+// The records of the delta rule with one decay per head, by runs of four rows of a request (counted from its first row of the
+// step). With P_i the product of the decays from the run's first row to row i, R_im = g_i ... g_(i-m+1), and A the state in
+// front of the run,
+//   d_i = beta_i (v_i - P_i A^T k_i - sum_m R_im (k_(i-m) . k_i) d_(i-m)),
+//   o_i = P_i A^T q_i + (k_i . q_i) d_i + sum_m R_im (k_(i-m) . q_i) d_(i-m),      m = 1 .. i's place in its run,
+// so everything a run needs of the state are eight dot products with A that do not wait for one another; what is left between
+// its rows are numbers that no column of the state enters, and they are formed here. Record: keys [D] (unit), queries [D] (unit,
+// times q_scale), beta, P, R_1..3, R_m (k . k) 1..3, k . q, R_m (k . q) 1..3, padding.
+constexpr int kDeltaScalars = 12;
+
+__global__ void delta_head_prepare_kernel(ScanArgs a) {
+  pdl_start();
+  const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
+  if (warp >= a.tokens * a.H) return;
+  const int t = warp / a.H, h = warp - t * a.H, D = a.D;
+  const int g = h / (a.H / a.G);
+  const int req = a.token_req[t];
+  const int place = req >= 0 ? (t - a.cu_seqlens[req]) & 3 : 0;      // the row's place in its run
+  const float* k_row = a.qkv + (size_t)t * a.ld_qkv + a.k_off + g * D;
+  const float* q_row = a.qkv + (size_t)t * a.ld_qkv + a.q_off + g * D;
+  float* rec = a.prep + ((size_t)t * a.H + h) * a.rec;
+  float k2 = 0.f, q2 = 0.f, kq = 0.f, n2[3] = {0.f, 0.f, 0.f}, kk[3] = {0.f, 0.f, 0.f}, kqs[3] = {0.f, 0.f, 0.f};
+  for (int d = lane; d < D; d += 32) {
+    const float k = k_row[d], q = q_row[d];
+    k2 += k * k, q2 += q * q, kq += k * q;
+#pragma unroll
+    for (int m = 0; m < 3; ++m)
+      if (m < place) {
+        const float b = k_row[d - (ptrdiff_t)(m + 1) * a.ld_qkv];
+        n2[m] += b * b, kk[m] += b * k, kqs[m] += b * q;
+      }
+  }
+  k2 = warp_sum(k2), q2 = warp_sum(q2), kq = warp_sum(kq);
+#pragma unroll
+  for (int m = 0; m < 3; ++m)
+    if (m < place) n2[m] = warp_sum(n2[m]), kk[m] = warp_sum(kk[m]), kqs[m] = warp_sum(kqs[m]);
+  const float kn = 1.f / sqrtf(k2 + 1e-6f), qn = a.q_scale / sqrtf(q2 + 1e-6f);
+  for (int d = lane; d < D; d += 32) {
+    rec[d] = k_row[d] * kn;
+    rec[D + d] = q_row[d] * qn;
+  }
+  float decay = 1.f;                     // lane m: the decay of the row m rows up, of the same run
+  if (lane <= place) {
+    const float rate = expf(load_as_f32(a.p1, a.p_dtype, h));
+    decay = expf(-rate * softplus_f(a.gates[(size_t)(t - lane) * a.ld_gates + a.f_off + h] + load_as_f32(a.p0, a.p_dtype, h)));
+  }
+  float R[4];
+  R[0] = __shfl_sync(0xffffffffu, decay, 0);
+#pragma unroll
+  for (int m = 1; m < 4; ++m) R[m] = R[m - 1] * __shfl_sync(0xffffffffu, decay, m);     // (one beyond the run's first row)
+  if (lane == 0) {
+    float* s = rec + 2 * D;
+    s[0] = 1.f / (1.f + expf(-a.gates[(size_t)t * a.ld_gates + a.i_off + h]));
+    s[1] = R[3];
+    s[8] = kq * kn * qn;
+#pragma unroll
+    for (int m = 0; m < 3; ++m) {
+      const float bn = m < place ? R[m] / sqrtf(n2[m] + 1e-6f) : 0.f;
+      s[2 + m] = R[m];
+      s[5 + m] = kk[m] * bn * kn;
+      s[9 + m] = kqs[m] * bn * qn;
+    }
   }
 }
 
@@ -363,12 +435,139 @@ __global__ void __launch_bounds__(kThreads) recurrent_scan_kernel(ScanArgs a, in
   if (kMode == kMatrixMemory && blockIdx.z == 0 && threadIdx.x == 0) fresh[(size_t)D * V + D] = m;
 }
 
-// out[t, h, c] = o[t, h, c] * rsqrt(mean_c o[t, h, :]^2 + eps) * w[h * w_stride + c] * sigmoid(gate[t, h, c]) * scale:
+// The scan of the delta rule with one decay per head: blocks and staging as above, the request's rows four at a time (see
+// delta_head_prepare_kernel); what is left over one at a time.
+template <int kLanes, int R, bool kVec4>
+__global__ void __launch_bounds__(kThreads) delta_head_scan_kernel(ScanArgs a, int chunk) {
+  pdl_wait();    // (no early trigger, as above)
+  extern __shared__ __align__(16) float stage[];
+  constexpr int kCols = kThreads / kLanes;
+  const int b = blockIdx.x, h = blockIdx.y;
+  const int start = a.cu_seqlens[b], n_rows = a.cu_seqlens[b + 1] - start;
+  if (n_rows <= 0 || a.token_req[start] < 0) return;
+  const int j = threadIdx.x % kLanes, cl = threadIdx.x / kLanes;
+  const int c = blockIdx.z * kCols + cl;
+  const bool col = c < a.V;
+  const int D = a.D, V = a.V, rec = a.rec;
+  const int phase = a.state_phase[b];
+  const float* old = a.state + (size_t)a.state_slots[b] * a.state_stride + ((size_t)phase * a.H + h) * D * V;
+  float* fresh = a.state + (size_t)a.state_slots[b] * a.state_stride + ((size_t)(1 - phase) * a.H + h) * D * V;
+  float C[R];
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int d = channel_of<kLanes, kVec4>(i, j);
+    C[i] = (col && d < D) ? old[(size_t)c * D + d] : 0.f;
+  }
+  const int buf_floats = chunk * (rec + kCols);
+  auto request = [&](int t0, int buf) {
+    const int n = min(chunk, n_rows - t0), rec4 = rec / 4;
+    float* st = stage + (size_t)buf * buf_floats;
+    float* vl = st + (size_t)chunk * rec;
+    for (int i = threadIdx.x; i < n * rec4; i += kThreads) {
+      const int tt = i / rec4, e = (i - tt * rec4) * 4;
+      cp_async<16>(st + (size_t)tt * rec + e, a.prep + ((size_t)(start + t0 + tt) * a.H + h) * rec + e);
+    }
+    for (int i = threadIdx.x; i < n * kCols; i += kThreads) {
+      const int tt = i / kCols, cc = blockIdx.z * kCols + (i - tt * kCols);
+      if (cc < V) cp_async<4>(vl + i, a.qkv + (size_t)(start + t0 + tt) * a.ld_qkv + a.v_off + h * V + cc);
+      else vl[i] = 0.f;
+    }
+    asm volatile("cp.async.commit_group;\n" ::: "memory");
+  };
+  request(0, 0);
+  int turn = 0;
+  for (int t0 = 0; t0 < n_rows; t0 += chunk, turn ^= 1) {      // chunk: a multiple of four, so that runs do not straddle it
+    const int n = min(chunk, n_rows - t0);
+    if (t0 + chunk < n_rows) {
+      request(t0 + chunk, turn ^ 1);
+      asm volatile("cp.async.wait_group 1;\n" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+    }
+    __syncthreads();
+    const float* stage_now = stage + (size_t)turn * buf_floats;
+    const float* vals = stage_now + (size_t)chunk * rec;
+    int tt = 0;
+    for (; tt + 3 < n; tt += 4) {
+      float k[4][R], ak[4], aq[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const float* r = stage_now + (size_t)(tt + u) * rec;
+        float q[R];
+        load_channels<kLanes, R, kVec4>(k[u], r, D, j);
+        load_channels<kLanes, R, kVec4>(q, r + D, D, j);
+        float pk[2] = {0.f, 0.f}, pq[2] = {0.f, 0.f};
+#pragma unroll
+        for (int i = 0; i < R; ++i) {
+          pk[i & 1] += C[i] * k[u][i];
+          pq[i & 1] += C[i] * q[i];
+        }
+        ak[u] = pk[0] + pk[1], aq[u] = pq[0] + pq[1];
+      }
+#pragma unroll
+      for (int u = 0; u < 4; ++u) ak[u] = lanes_sum<kLanes>(ak[u]), aq[u] = lanes_sum<kLanes>(aq[u]);
+      float d[4], o[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const float* s = stage_now + (size_t)(tt + u) * rec + 2 * D;
+        float want = vals[(tt + u) * kCols + cl] - s[1] * ak[u];
+        o[u] = s[1] * aq[u];
+#pragma unroll
+        for (int m = 0; m < u; ++m) {
+          want -= s[5 + m] * d[u - 1 - m];
+          o[u] += s[9 + m] * d[u - 1 - m];
+        }
+        d[u] = s[0] * want;
+        o[u] += s[8] * d[u];
+      }
+      const float* last = stage_now + (size_t)(tt + 3) * rec + 2 * D;
+      const float keep = last[1], w0 = d[0] * last[4], w1 = d[1] * last[3], w2 = d[2] * last[2];
+#pragma unroll
+      for (int i = 0; i < R; ++i) C[i] = keep * C[i] + ((k[0][i] * w0 + k[1][i] * w1) + (k[2][i] * w2 + k[3][i] * d[3]));
+      if (j == 0 && col) {
+        float* o_row = a.out + (size_t)(start + t0 + tt) * a.ld_out + (size_t)h * V + c;
+#pragma unroll
+        for (int u = 0; u < 4; ++u) o_row[(size_t)u * a.ld_out] = o[u];
+      }
+    }
+    for (; tt < n; ++tt) {
+      const float* r = stage_now + (size_t)tt * rec;
+      const float beta = r[2 * D], g = r[2 * D + 2];
+      float k[R], q[R];
+      load_channels<kLanes, R, kVec4>(k, r, D, j);
+      load_channels<kLanes, R, kVec4>(q, r + D, D, j);
+      float kv[2] = {0.f, 0.f};
+#pragma unroll
+      for (int i = 0; i < R; ++i) {
+        C[i] *= g;
+        kv[i & 1] += C[i] * k[i];
+      }
+      const float dlt = beta * (vals[tt * kCols + cl] - lanes_sum<kLanes>(kv[0] + kv[1]));
+      float num[2] = {0.f, 0.f};
+#pragma unroll
+      for (int i = 0; i < R; ++i) {
+        C[i] += k[i] * dlt;
+        num[i & 1] += C[i] * q[i];
+      }
+      const float o = lanes_sum<kLanes>(num[0] + num[1]);
+      if (j == 0 && col) a.out[(size_t)(start + t0 + tt) * a.ld_out + (size_t)h * V + c] = o;
+    }
+    __syncthreads();                           // everyone has read this buffer before the chunk after next is requested into it
+  }
+#pragma unroll
+  for (int i = 0; i < R; ++i) {
+    const int d = channel_of<kLanes, kVec4>(i, j);
+    if (col && d < D) fresh[(size_t)c * D + d] = C[i];
+  }
+}
+
+// out[t, h, c] = o[t, h, c] * rsqrt(mean_c o[t, h, :]^2 + eps) * w[h * w_stride + c] * act(gate[t, h, c]) * scale, act the
+// sigmoid (gate_act OI_ACT_NONE) or silu (OI_ACT_SILU):
 // the per-head unit norm, the weight and the output gate of a recurrent mixer, one warp per (row, head).
 template <typename TO>
 __global__ void head_norm_gate_kernel(TO* __restrict__ out, long long ld_out, const float* __restrict__ o, long long ld_o,
                                       const float* __restrict__ gate, long long ld_gate, const void* __restrict__ w,
-                                      int w_dtype, int w_stride, int tokens, int H, int V, float eps, float scale) {
+                                      int w_dtype, int w_stride, int tokens, int H, int V, float eps, float scale, int gate_act) {
   pdl_start();
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (warp >= tokens * H) return;
@@ -380,7 +579,7 @@ __global__ void head_norm_gate_kernel(TO* __restrict__ out, long long ld_out, co
   const float r = 1.f / sqrtf(ss / (float)V + eps);
   for (int c = lane; c < V; c += 32) {
     const float gz = gate[(size_t)t * ld_gate + (size_t)h * V + c];
-    const float val = row[c] * r * load_as_f32(w, w_dtype, (size_t)h * w_stride + c) * (1.f / (1.f + expf(-gz))) * scale;
+    const float val = row[c] * r * load_as_f32(w, w_dtype, (size_t)h * w_stride + c) * gate_value(gz, gate_act) * scale;
     out[(size_t)t * ld_out + (size_t)h * V + c] = from_f32<TO>(val);
   }
 }
@@ -389,7 +588,7 @@ __global__ void head_norm_gate_kernel(TO* __restrict__ out, long long ld_out, co
 template <typename TO>
 __global__ void row_norm_gate_kernel(TO* __restrict__ out, long long ld_out, const float* __restrict__ o, long long ld_o,
                                      const float* __restrict__ gate, long long ld_gate, const void* __restrict__ w, int w_dtype,
-                                     int V, float eps, float scale) {
+                                     int V, float eps, float scale, int gate_act) {
   pdl_start();
   __shared__ float red[32];
   const int t = blockIdx.x;
@@ -400,17 +599,19 @@ __global__ void row_norm_gate_kernel(TO* __restrict__ out, long long ld_out, con
   const float r = 1.f / sqrtf(ss / (float)V + eps);
   for (int c = threadIdx.x; c < V; c += blockDim.x) {
     const float gz = gate[(size_t)t * ld_gate + c];
-    out[(size_t)t * ld_out + c] = from_f32<TO>(row[c] * r * load_as_f32(w, w_dtype, c) * (1.f / (1.f + expf(-gz))) * scale);
+    out[(size_t)t * ld_out + c] = from_f32<TO>(row[c] * r * load_as_f32(w, w_dtype, c) * gate_value(gz, gate_act) * scale);
   }
 }
 
 }  // namespace
 
 // floats of scratch the scan wants per row: oi_recurrent_scan's `prep` is [tokens, H, that]
-OI_API int oi_recurrent_record(int D) { return (3 * D + 2 + 3) & ~3; }   // a multiple of four floats: 16-byte copies
+OI_API int oi_recurrent_record(int mode, int D) {                        // a multiple of four floats: 16-byte copies
+  return mode == kDeltaHeadDecay ? (2 * D + kDeltaScalars + 3) & ~3 : (3 * D + 2 + 3) & ~3;
+}
 
 // mode 0: matrix memory (p0, p1: the two gate biases [H]); mode 1: gated delta rule (p0: dt [H * D], p1: A [H];
-// decay: a [tokens, ld_decay]); mode 2: linear attention with a fixed decay per head (p0: lambda [H]; qkv is written: the
+// decay: a [tokens, ld_decay]); mode 3: the delta rule with one decay per head (a at f_off of `gates`, p0: dt [H], p1: A [H]); mode 2: linear attention with a fixed decay per head (p0: lambda [H]; qkv is written: the
 // values get their silu in place). State: [slots][2][H][D * V (+ D + 1 in mode 0)] floats. prep: scratch, see above.
 OI_API int oi_recurrent_scan(int mode, const float* qkv, long long ld_qkv, int q_off, int k_off, int v_off, const float* gates,
                              long long ld_gates, int i_off, int f_off, const float* decay, long long ld_decay, const void* p0,
@@ -418,7 +619,7 @@ OI_API int oi_recurrent_scan(int mode, const float* qkv, long long ld_qkv, int q
                              long long state_stride, const int* cu_seqlens, const int* token_req, const int* state_slots,
                              const int* state_phase, float* out, long long ld_out, int tokens, int requests, int H, int G, int D,
                              int V, void* stream) {
-  OI_REQUIRE(mode == kMatrixMemory || mode == kGatedDelta || mode == kLinearDecay, "recurrent_scan: unknown mode %d", mode);
+  OI_REQUIRE(mode == kMatrixMemory || mode == kGatedDelta || mode == kLinearDecay || mode == kDeltaHeadDecay, "recurrent_scan: unknown mode %d", mode);
   OI_REQUIRE(requests >= 0 && tokens >= 0 && H > 0 && G > 0 && H % G == 0 && D > 0 && V > 0,
              "recurrent_scan: bad sizes H=%d G=%d D=%d V=%d", H, G, D, V);
   OI_REQUIRE(D <= 32 * kMaxRegs, "recurrent_scan: %d key channels per head, at most %d", D, 32 * kMaxRegs);
@@ -431,7 +632,7 @@ OI_API int oi_recurrent_scan(int mode, const float* qkv, long long ld_qkv, int q
   a.qkv = qkv, a.ld_qkv = ld_qkv, a.q_off = q_off, a.k_off = k_off, a.v_off = v_off;
   a.gates = gates, a.ld_gates = ld_gates, a.i_off = i_off, a.f_off = f_off;
   a.decay = decay, a.ld_decay = ld_decay, a.p0 = p0, a.p1 = p1, a.p_dtype = p_dtype, a.cap = cap, a.q_scale = q_scale;
-  a.prep = prep, a.rec = oi_recurrent_record(D);
+  a.prep = prep, a.rec = oi_recurrent_record(mode, D);
   a.state = state, a.state_stride = state_stride, a.cu_seqlens = cu_seqlens, a.token_req = token_req;
   a.state_slots = state_slots, a.state_phase = state_phase, a.out = out, a.ld_out = ld_out;
   a.tokens = tokens, a.H = H, a.G = G, a.D = D, a.V = V;
@@ -439,8 +640,30 @@ OI_API int oi_recurrent_scan(int mode, const float* qkv, long long ld_qkv, int q
   const int warps = tokens * H;
   if (mode == kMatrixMemory) oi_launch(recurrent_prepare_kernel<kMatrixMemory>, (warps + 3) / 4, 128, 0, s, a);
   else if (mode == kLinearDecay) oi_launch(recurrent_prepare_kernel<kLinearDecay>, (warps + 3) / 4, 128, 0, s, a);
+  else if (mode == kDeltaHeadDecay) oi_launch(delta_head_prepare_kernel, (warps + 3) / 4, 128, 0, s, a);
   else oi_launch(recurrent_prepare_kernel<kGatedDelta>, (warps + 3) / 4, 128, 0, s, a);
   OI_CHECK_LAUNCH();
+  if (mode == kDeltaHeadDecay) {
+    const int rows = D <= 128 ? 16 : (D <= 256 ? 8 : 4);       // per buffer: two buffers of at most 19 KB
+#define OI_DELTA_HEAD(LANES, REGS)                                                                                          \
+  do {                                                                                                                      \
+    constexpr int cols = kThreads / LANES;                                                                                  \
+    const dim3 grid(requests, H, (V + cols - 1) / cols);                                                                    \
+    const size_t smem = 2 * (size_t)rows * (a.rec + cols) * sizeof(float);                                                  \
+    oi_fence_next_launch();      /* plain stream order, as below */                                                         \
+    if (D % 4 == 0) oi_launch(delta_head_scan_kernel<LANES, REGS, true>, grid, kThreads, smem, s, a, rows);                 \
+    else oi_launch(delta_head_scan_kernel<LANES, REGS, false>, grid, kThreads, smem, s, a, rows);                           \
+  } while (0)
+    if (D <= 16) OI_DELTA_HEAD(4, 4);
+    else if (D <= 32) OI_DELTA_HEAD(8, 4);
+    else if (D <= 64) OI_DELTA_HEAD(8, 8);
+    else if (D <= 128) OI_DELTA_HEAD(8, 16);
+    else if (D <= 256) OI_DELTA_HEAD(16, 16);
+    else OI_DELTA_HEAD(32, 16);
+#undef OI_DELTA_HEAD
+    OI_CHECK_LAUNCH();
+    return OI_OK;
+  }
   // rows per buffer: two buffers of at most 13 KB; the linear decay, which walks four rows at a time, takes more (up to 44 KB)
   const int chunk = mode == kLinearDecay ? (D <= 64 ? 24 : (D <= 128 ? 12 : (D <= 256 ? 4 : 2)))
                                          : (D <= 64 ? 16 : (D <= 128 ? 8 : (D <= 256 ? 4 : 2)));
@@ -484,24 +707,24 @@ OI_API int oi_recurrent_scan(int mode, const float* qkv, long long ld_qkv, int q
 
 OI_API int oi_head_norm_gate(void* out, int out_dtype, long long ld_out, const float* o, long long ld_o, const float* gate,
                              long long ld_gate, const void* w, int w_dtype, int w_stride, int tokens, int H, int V, float eps,
-                             float scale, void* stream) {
-  OI_REQUIRE(tokens >= 0 && H > 0 && V > 0, "head_norm_gate: bad sizes");
+                             float scale, int gate_act, void* stream) {
+  OI_REQUIRE(tokens >= 0 && H > 0 && V > 0 && (gate_act == OI_ACT_NONE || gate_act == OI_ACT_SILU), "head_norm_gate: bad sizes or gate");
   if (tokens == 0) return OI_OK;
   const int warps = tokens * H, blocks = (warps + 7) / 8;
   cudaStream_t s = (cudaStream_t)stream;
   if (H == 1 && V >= 256 && (out_dtype == OI_F32 || out_dtype == OI_BF16)) {     // one long row: a block a row, not a warp
     const int threads = V >= 1024 ? 256 : 128;
     if (out_dtype == OI_F32)
-      oi_launch(row_norm_gate_kernel<float>, tokens, threads, 0, s, (float*)out, ld_out, o, ld_o, gate, ld_gate, w, w_dtype, V, eps, scale);
+      oi_launch(row_norm_gate_kernel<float>, tokens, threads, 0, s, (float*)out, ld_out, o, ld_o, gate, ld_gate, w, w_dtype, V, eps, scale, gate_act);
     else
-      oi_launch(row_norm_gate_kernel<bf16>, tokens, threads, 0, s, (bf16*)out, ld_out, o, ld_o, gate, ld_gate, w, w_dtype, V, eps, scale);
+      oi_launch(row_norm_gate_kernel<bf16>, tokens, threads, 0, s, (bf16*)out, ld_out, o, ld_o, gate, ld_gate, w, w_dtype, V, eps, scale, gate_act);
     OI_CHECK_LAUNCH();
     return OI_OK;
   }
   if (out_dtype == OI_F32)
-    oi_launch(head_norm_gate_kernel<float>, blocks, 256, 0, s, (float*)out, ld_out, o, ld_o, gate, ld_gate, w, w_dtype, w_stride, tokens, H, V, eps, scale);
+    oi_launch(head_norm_gate_kernel<float>, blocks, 256, 0, s, (float*)out, ld_out, o, ld_o, gate, ld_gate, w, w_dtype, w_stride, tokens, H, V, eps, scale, gate_act);
   else if (out_dtype == OI_BF16)
-    oi_launch(head_norm_gate_kernel<bf16>, blocks, 256, 0, s, (bf16*)out, ld_out, o, ld_o, gate, ld_gate, w, w_dtype, w_stride, tokens, H, V, eps, scale);
+    oi_launch(head_norm_gate_kernel<bf16>, blocks, 256, 0, s, (bf16*)out, ld_out, o, ld_o, gate, ld_gate, w, w_dtype, w_stride, tokens, H, V, eps, scale, gate_act);
   else
     OI_REQUIRE(false, "head_norm_gate: unknown dtype code %d", out_dtype);
   OI_CHECK_LAUNCH();

@@ -177,13 +177,22 @@ class AttentionPlan:
     decode_merge_in_kernel: bool = False
 
 
+def first_visible(pos: int, window: Optional[int]) -> int:
+    """The first key a query at ``pos`` sees. window None or 0: every key; > 0: the last ``window`` keys; < 0: the keys of
+    its own chunk of -window positions."""
+    if not window:
+        return 0
+    return max(0, pos - window + 1) if window > 0 else pos - pos % -window
+
+
 def decode_splits(num_rows: int, nkv: int, sm_count: int, max_kv_len: Optional[int], capacity: Optional[int] = None,
-                  long_ok: bool = True) -> int:
+                  long_ok: bool = True, chunk: int = 0) -> int:
     """Slices per decode row: as many as fill the GPU once (two CTAs of four slices per SM), a
     multiple of four, each at least 32 keys long when the lengths are known. ``capacity``: the keys a row
     may hold when the lengths are not known (a recorded step: the width of its block table). ``long_ok`` False: no
     more slices than a cluster merges, whatever the lengths (steps that also bring prompt portions: the scratch of
-    slices merged by the second kernel is indexed by the step's rows, and the GPU is busy anyway)."""
+    slices merged by the second kernel is indexed by the step's rows, and the GPU is busy anyway). ``chunk``: a row never
+    sees more keys than that."""
     if policy.batch_invariant():
         return policy.INVARIANT_DECODE_SPLITS      # the same cutting whatever else is in the step
     pairs = max(1, num_rows * nkv)
@@ -196,6 +205,8 @@ def decode_splits(num_rows: int, nkv: int, sm_count: int, max_kv_len: Optional[i
     ns = min(ns, limit)
     if ns > DECODE_MAX_SPLITS:
         ns = 1 << (ns.bit_length() - 1)    # beyond what a cluster merges: 64 or 128 (72 slices measured slower than 64)
+    if chunk > 0:
+        max_kv_len = min(chunk, max_kv_len) if max_kv_len is not None else chunk
     if max_kv_len is not None:
         ns = min(ns, max(DECODE_WARPS, (max_kv_len // DECODE_MIN_KEYS_PER_SPLIT) // DECODE_WARPS * DECODE_WARPS))
     return ns
@@ -236,13 +247,14 @@ def plan_items(q_lens, kv_lens, group: int, nkv: int, window: Optional[int], sm_
         for t0 in range(0, n, tpt):
             toks = min(tpt, n - t0)
             pos0 = kv - n + t0
-            lo = (max(0, pos0 - window + 1) if window else 0) & ~(KEYS_PER_TILE - 1)
+            lo = first_visible(pos0, window) & ~(KEYS_PER_TILE - 1)
             span_tiles = -(-(pos0 + toks - lo) // KEYS_PER_TILE)
             tiles.append((b, t0, toks, span_tiles))
     max_splits = 1
     decode_items = []
     if decode_reqs:
-        ns = decode_splits(len(decode_reqs), nkv, sm_count, max(kv_lens[b] for b in decode_reqs), long_ok=not tiles)
+        ns = decode_splits(len(decode_reqs), nkv, sm_count, max(kv_lens[b] for b in decode_reqs), long_ok=not tiles,
+                           chunk=-window if window and window < 0 else 0)
         max_splits = ns
         for b in decode_reqs:
             row_splits[starts[b]] = ns
@@ -266,13 +278,14 @@ def plan_items(q_lens, kv_lens, group: int, nkv: int, window: Optional[int], sm_
             row_splits, max_splits, tile_split)
 
 
-def plan_items_static_decode(num_requests: int, group: int, nkv: int, sm_count: int, capacity: Optional[int] = None):
+def plan_items_static_decode(num_requests: int, group: int, nkv: int, sm_count: int, capacity: Optional[int] = None,
+                             chunk: int = 0):
     """Items of a decode step whose launch is recorded once and replayed (a CUDA graph): one
     query token per request, and a number of key slices that depends on the batch size only;
     the kernels find each slice's bounds from the request's current length."""
     empty = np.zeros((0, 4), dtype=np.int32)
     if group <= DECODE_MAX_GROUP:
-        ns = decode_splits(num_requests, nkv, sm_count, None, capacity)
+        ns = decode_splits(num_requests, nkv, sm_count, None, capacity, chunk=chunk)
         items = np.asarray([(b, 0, s0, ns) for b in range(num_requests) for s0 in range(0, ns, DECODE_WARPS)],
                            dtype=np.int32).reshape(-1, 4)
         return empty, items, np.full(num_requests, ns, dtype=np.int32), ns, False
@@ -295,7 +308,7 @@ def _plan_for(ctx, group_step, group: int, nq: int, nkv: int, hd: int, window, d
             table = getattr(group_step, "block_table", None)
             capacity = int(table.shape[1]) * ctx.cache.page_size if table is not None and table.dim() == 2 else None
             t_items, d_items, row_splits, max_splits, tile_split = plan_items_static_decode(
-                ctx.num_requests, group, nkv, _sm_count(device), capacity)
+                ctx.num_requests, group, nkv, _sm_count(device), capacity, chunk=-window if window and window < 0 else 0)
         else:
             rows = tile_rows(ctx.q_lens_host, group)
             page = ctx.cache.page_size

@@ -58,11 +58,16 @@ _SIGNATURES = {
     "oi_latent_store": [P, L, I, I, P, L, I, P, I, P, I, I, F, F, P],
     "oi_head_gate": [P, L, P, L, I, I, I, I, P],
     "oi_xielu": [P, P, I, P, I, L, P],
-    "oi_short_conv_strided": [P, I, L, P, I, L, P, I, P, L, P, P, P, P, I, I, I, I, I, I, I, P],
+    "oi_short_conv_strided": [P, I, L, P, I, L, P, I, P, L, P, P, P, P, I, I, I, I, I, I, I, P, P, P],
+    "oi_layernorm_cast": [P, I, P, I, P, I, P, I, I, F, F, P],
+    "oi_branch_join": [P, P, P, P, P, F, F, F, P, I, F, P, P, I, I, P],
+    "oi_joint_norm_half_store": [P, I, L, I, I, I, I, I, P, P, P, F, P, P, I, I, P, P, P, P, L, I, P],
+    "oi_rglru_gates": [P, L, P, I, P, P, P, L, I, P, L, P, P, I, L, P, L, P, P, P, I, I, I, P],
+    "oi_affine_scan": [P, I, L, P, L, I, P, L, P, P, L, P, P, P, I, I, I, P],
     "oi_glu_act": [P, P, I, I, I, I, I, F, P],
     "oi_recurrent_scan": [I, P, L, I, I, I, P, L, I, I, P, L, P, P, I, F, F, P, P, L, P, P, P, P, P, L, I, I, I, I, I, I, P],
-    "oi_recurrent_record": [I],
-    "oi_head_norm_gate": [P, I, L, P, L, P, L, P, I, I, I, I, I, F, F, P],
+    "oi_recurrent_record": [I, I],
+    "oi_head_norm_gate": [P, I, L, P, L, P, L, P, I, I, I, I, I, F, F, I, P],
     "oi_hyper_step": [P, I, I, I, P, P, F, F, P, P, P, I, P, I, F, F, P, I, P, P],
     "oi_hyper_fanout": [P, P, I, I, I, I, P],
     "oi_scaled_sum": [P, P, P, F, F, L, P],
@@ -70,7 +75,7 @@ _SIGNATURES = {
     "oi_moe_route": [P, I, L, P, I, I, I, I, I, P, P, P, P, P],
     "oi_moe_experts": [P, I, L, P, P, I, I, I, I, I, F, I, P, P, P, P, P, P, P, P, P],
     "oi_moe_route_table": [P, P, I, I, I, I, P, P, P, P, P],
-    "oi_moe_route_scored": [P, I, L, P, I, I, I, I, I, I, P, I, I, P, P, P, P, P],
+    "oi_moe_route_scored": [P, I, L, P, I, I, I, I, I, I, I, P, I, I, F, P, P, P, P, P],
     "oi_dyt_step": [P, P, P, P, P, I, P, P, P, I, P, I, P, I, I, P],
     "oi_rope_norm_store": [P, I, L, I, I, I, I, I, P, I, L, P, P, I, I, I, F, P, P, P, P, L, I, I, P],
     "oi_moe_small": [I, I],

@@ -5,7 +5,7 @@ the current stream. None of them has another implementation to fall back to.
 """
 from __future__ import annotations
 
-from typing import Optional
+from typing import NamedTuple, Optional
 
 import torch
 
@@ -350,9 +350,9 @@ def sample(out: torch.Tensor, logits: torch.Tensor, probs_scratch: torch.Tensor,
 # layers with a 32-bit residual stream (csrc/branch_ops.cu)
 # ---------------------------------------------------------------------------
 def rmsnorm_cast(out: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, eps: float, *,
-                 row_idx: Optional[torch.Tensor] = None, weight_offset: float = 0.0) -> torch.Tensor:
+                 row_idx: Optional[torch.Tensor] = None, weight_offset: float = 0.0, center: bool = False) -> torch.Tensor:
     """out = x * rsqrt(mean(x^2) + eps) * (weight_offset + weight) row by row, where x and out may differ in
-    type (a float32 stream normed into the model's type). ``row_idx``: output row r reads x[row_idx[r]]."""
+    type (a float32 stream normed into the model's type). ``center``: a layer norm, the row's mean is taken off first. ``row_idx``: output row r reads x[row_idx[r]]."""
     _cuda(out, x, weight, row_idx)
     _i32(row_idx, "rmsnorm_cast row_idx")
     hidden, rows = x.shape[-1], out.shape[0]
@@ -361,9 +361,46 @@ def rmsnorm_cast(out: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, eps: 
         raise KernelError(f"rmsnorm_cast: shapes x={tuple(x.shape)} out={tuple(out.shape)} weight={tuple(weight.shape)}")
     if (row_idx is None and rows != x.shape[0]) or (row_idx is not None and row_idx.numel() != rows):
         raise KernelError("rmsnorm_cast: row counts do not match")
-    _lib.check(_lib.load().oi_rmsnorm_cast(out.data_ptr(), _code(out, "rmsnorm_cast"), x.data_ptr(), _code(x, "rmsnorm_cast"),
-                                           weight.data_ptr(), _code(weight, "rmsnorm_cast weight"), _ptr(row_idx), rows,
-                                           hidden, float(eps), float(weight_offset), _stream()), "rmsnorm_cast")
+    lib = _lib.load()
+    fn = lib.oi_layernorm_cast if center else lib.oi_rmsnorm_cast
+    _lib.check(fn(out.data_ptr(), _code(out, "rmsnorm_cast"), x.data_ptr(), _code(x, "rmsnorm_cast"), weight.data_ptr(),
+                  _code(weight, "rmsnorm_cast weight"), _ptr(row_idx), rows, hidden, float(eps), float(weight_offset), _stream()), "rmsnorm_cast")
+    return out
+
+
+class NormedPair(NamedTuple):
+    """Two results [tokens, width] that were computed side by side: ca rms(a; wa) + cb rms(b; wb)."""
+
+    a: torch.Tensor
+    b: torch.Tensor
+    wa: torch.Tensor
+    wb: torch.Tensor
+    ca: float
+    cb: float
+    eps: float
+
+
+def branch_join(h: Optional[torch.Tensor], branch, *, weight: Optional[torch.Tensor] = None, center: bool = False, eps: float = 0.0,
+                low: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """h += norm(v) and ``low`` = the new h in bfloat16 (h float32 rows, or None), ``out`` = norm(v), where v is ``branch``
+    (float32 [tokens, width]) or the sum a ``NormedPair`` stands for, and norm a layer norm (``center``) or an RMS norm with
+    the float32 ``weight``; without a weight v as it is."""
+    pair = branch if isinstance(branch, NormedPair) else None
+    a, b = (pair.a, pair.b) if pair else (branch, None)
+    rows, width = a.shape
+    _cuda(h, a, b, weight, low, out, *((pair.wa, pair.wb) if pair else ()))
+    for t in (h, a, b, out):
+        if t is not None and (t.dtype != torch.float32 or t.shape != (rows, width) or not t.is_contiguous()):
+            raise KernelError("branch_join: the stream and the branches must be contiguous float32 rows of one shape")
+    for w in ((weight,) + ((pair.wa, pair.wb) if pair else ())):
+        if w is not None and (w.dtype != torch.float32 or w.numel() != width or not w.is_contiguous()):
+            raise KernelError("branch_join: a weight must be float32 of the stream's width")
+    if low is not None and (h is None or low.dtype != torch.bfloat16 or low.shape != (rows, width) or not low.is_contiguous()):
+        raise KernelError("branch_join: low is the stream's bfloat16 copy")
+    _lib.check(_lib.load().oi_branch_join(
+        _ptr(h), a.data_ptr(), _ptr(b), _ptr(pair.wa) if pair else 0, _ptr(pair.wb) if pair else 0, float(pair.ca) if pair else 1.0,
+        float(pair.cb) if pair else 0.0, float(pair.eps) if pair else 0.0, _ptr(weight), 1 if center else 0, float(eps), _ptr(out),
+        _ptr(low), rows, width, _stream()), "branch_join")
     return out
 
 
@@ -499,10 +536,15 @@ def glu_code(name: str) -> int:
 
 def short_conv_act(out: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, state: Optional[torch.Tensor], cu_seqlens: torch.Tensor,
                    token_req: torch.Tensor, state_slots: torch.Tensor, state_phase: Optional[torch.Tensor], *, act: str = "none",
-                   add_input: bool = False) -> torch.Tensor:
+                   add_input: bool = False, in_bias: Optional[torch.Tensor] = None,
+                   out_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``short_conv`` on a slice of columns of wider buffers (x and out [tokens, channels] with free row strides) and
-    with an activation on the filter's result ("none" or "silu")."""
-    _cuda(out, x, weight, state, cu_seqlens, token_req, state_slots, state_phase)
+    with an activation on the filter's result ("none" or "silu"). ``in_bias`` / ``out_bias`` (float32 [channels]) are added to
+    every input (not to the zeros before a request's start) and to the filter's result."""
+    _cuda(out, x, weight, state, cu_seqlens, token_req, state_slots, state_phase, in_bias, out_bias)
+    for b in (in_bias, out_bias):
+        if b is not None and (b.dtype != torch.float32 or b.numel() != x.shape[1] or not b.is_contiguous()):
+            raise KernelError("short_conv_act: a bias must be contiguous float32 [channels]")
     tokens, channels = x.shape
     taps = weight.shape[1]
     if out.shape != x.shape or weight.shape[0] != channels or x.stride(1) != 1 or out.stride(1) != 1 or not weight.is_contiguous():
@@ -517,14 +559,14 @@ def short_conv_act(out: torch.Tensor, x: torch.Tensor, weight: torch.Tensor, sta
         out.data_ptr(), _code(out, "short_conv"), out.stride(0), x.data_ptr(), _code(x, "short_conv"), x.stride(0), weight.data_ptr(),
         _code(weight, "short_conv weight"), _ptr(state), stride, cu_seqlens.data_ptr(), token_req.data_ptr(), state_slots.data_ptr(),
         _ptr(state_phase), tokens, cu_seqlens.numel() - 1, channels, taps, 1 if add_input else 0, 1,
-        {"none": 0, "silu": 1}[act], _stream()), "short_conv_act")
+        {"none": 0, "silu": 1}[act], _ptr(in_bias), _ptr(out_bias), _stream()), "short_conv_act")
     return out
 
 
 # ---------------------------------------------------------------------------
 # recurrent mixers with a matrix memory per head (csrc/recurrent.cu)
 # ---------------------------------------------------------------------------
-SCAN_MATRIX_MEMORY, SCAN_GATED_DELTA, SCAN_LINEAR_DECAY = 0, 1, 2
+SCAN_MATRIX_MEMORY, SCAN_GATED_DELTA, SCAN_LINEAR_DECAY, SCAN_DELTA_HEAD_DECAY = 0, 1, 2, 3
 
 
 def recurrent_scan(mode: int, out: torch.Tensor, qkv: torch.Tensor, offsets, gates: torch.Tensor, gate_offsets, state: torch.Tensor,
@@ -545,7 +587,7 @@ def recurrent_scan(mode: int, out: torch.Tensor, qkv: torch.Tensor, offsets, gat
         raise KernelError(f"recurrent_scan: state {tuple(state.shape)} is not [slots, 2, {heads}, {elems}]")
     L = _lib.load()
     tokens = out.shape[0]
-    prep = torch.empty((tokens, heads, L.oi_recurrent_record(dim)), dtype=torch.float32, device=out.device)
+    prep = torch.empty((tokens, heads, L.oi_recurrent_record(mode, dim)), dtype=torch.float32, device=out.device)
     _lib.check(L.oi_recurrent_scan(
         mode, qkv.data_ptr(), qkv.stride(0), int(offsets[0]), int(offsets[1]), int(offsets[2]), gates.data_ptr(), gates.stride(0),
         int(gate_offsets[0]), int(gate_offsets[1]), _ptr(decay), 0 if decay is None else decay.stride(0), p0.data_ptr(), p1.data_ptr(),
@@ -556,8 +598,8 @@ def recurrent_scan(mode: int, out: torch.Tensor, qkv: torch.Tensor, offsets, gat
 
 
 def head_norm_gate(out: torch.Tensor, o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, heads: int, vdim: int, eps: float,
-                   *, weight_per_head: bool, scale: float = 1.0) -> torch.Tensor:
-    """out[t, h, :] = o[t, h, :] / rms(o[t, h, :]) * w * sigmoid(gate[t, h, :]) * scale; o and gate float32 rows,
+                   *, weight_per_head: bool, scale: float = 1.0, gate_act: str = "sigmoid") -> torch.Tensor:
+    """out[t, h, :] = o[t, h, :] / rms(o[t, h, :]) * w * act(gate[t, h, :]) * scale (``gate_act``: "sigmoid" or "silu"); o and gate float32 rows,
     ``weight`` [heads * vdim] (``weight_per_head``) or [vdim] shared by the heads."""
     _cuda(out, o, gate, weight)
     if o.dtype != torch.float32 or gate.dtype != torch.float32 or o.stride(1) != 1 or gate.stride(1) != 1 or out.stride(1) != 1 \
@@ -566,7 +608,7 @@ def head_norm_gate(out: torch.Tensor, o: torch.Tensor, gate: torch.Tensor, weigh
     _lib.check(_lib.load().oi_head_norm_gate(out.data_ptr(), _code(out, "head_norm_gate"), out.stride(0), o.data_ptr(), o.stride(0),
                                              gate.data_ptr(), gate.stride(0), weight.data_ptr(), _code(weight, "head_norm_gate weight"),
                                              vdim if weight_per_head else 0, o.shape[0], heads, vdim, float(eps), float(scale),
-                                             _stream()), "head_norm_gate")
+                                             {"sigmoid": 0, "silu": 1}[gate_act], _stream()), "head_norm_gate")
     return out
 
 
@@ -630,19 +672,23 @@ def scaled_sum(out: torch.Tensor, a: torch.Tensor, b: torch.Tensor, ca: float, c
 # routed experts (csrc/moe.cu)
 # ---------------------------------------------------------------------------
 def moe_route(x: torch.Tensor, w_router: torch.Tensor, top: int, *, scoring: str = "softmax_top",
-              correction: Optional[torch.Tensor] = None, groups: int = 1, keep_groups: int = 1):
+              correction: Optional[torch.Tensor] = None, groups: int = 1, keep_groups: int = 1, identity: int = 0,
+              weight_scale: float = 1.0):
     """Router logits in float32, the ``top`` largest per row and their softmax, and the rows grouped by expert.
     ``scoring`` "sigmoid_groups": scores sigmoid(logit); the choice goes by score + ``correction`` (float32 [experts]) among
     the experts of the ``keep_groups`` best of ``groups`` equal groups of neighbours (a group's score: the sum of its two
-    largest choice scores); the weights are the chosen scores divided by their sum.
+    largest choice scores); the weights are the chosen scores divided by their sum. "softmax_groups": softmax scores, a
+    group's score is its largest choice score, the weights are the chosen scores times ``weight_scale``. The last ``identity``
+    rows of the router (and of the correction and the groups) are choices without an expert.
     Returns (ids [rows, top] int32, weights [rows, top] float32, sorted pairs, tile list): the last two feed ``moe_experts``."""
     _cuda(x, w_router, correction)
-    if scoring not in ("softmax_top", "sigmoid_groups"):
+    codes = {"softmax_top": 0, "sigmoid_groups": 1, "softmax_groups": 2}
+    if scoring not in codes:
         raise KernelError(f"moe_route: unknown scoring {scoring!r}")
     if correction is not None and (correction.dtype != torch.float32 or correction.numel() != w_router.shape[0] or not correction.is_contiguous()):
         raise KernelError("moe_route: the correction must be a contiguous float32 tensor of one number an expert")
     rows, K = x.shape
-    E = w_router.shape[0]
+    E = w_router.shape[0] - identity
     if x.stride(1) != 1 or not w_router.is_contiguous() or w_router.shape[1] != K:
         raise KernelError(f"moe_route: x={tuple(x.shape)} router={tuple(w_router.shape)}")
     L = _lib.load()
@@ -651,8 +697,8 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, top: int, *, scoring: str
     order = torch.empty(rows * top, dtype=torch.int32, device=x.device)
     tiles = torch.empty(3 * L.oi_moe_max_tiles(rows * top, E) + 1, dtype=torch.int32, device=x.device)
     _lib.check(L.oi_moe_route_scored(x.data_ptr(), _code(x, "moe_route"), x.stride(0), w_router.data_ptr(),
-                                     _code(w_router, "moe_route router"), rows, K, E, int(top), 1 if scoring == "sigmoid_groups" else 0,
-                                     _ptr(correction), int(groups), int(keep_groups), ids.data_ptr(), wts.data_ptr(), order.data_ptr(),
+                                     _code(w_router, "moe_route router"), rows, K, E, int(identity), int(top), codes[scoring],
+                                     _ptr(correction), int(groups), int(keep_groups), float(weight_scale), ids.data_ptr(), wts.data_ptr(), order.data_ptr(),
                                      tiles.data_ptr(), _stream()), "moe_route")
     return ids, wts, order, tiles
 
@@ -858,4 +904,67 @@ def mingru_scan(out: torch.Tensor, zug: torch.Tensor, col_step: int, bias: torch
         state.data_ptr(), state.stride(0), ctx.cu_seqlens.data_ptr(), ctx.token_req.data_ptr(), ctx.state_slots.data_ptr(),
         out.shape[0], ctx.num_requests, C, 1 if ctx.decode_only or 1 in ctx.q_lens_host else 0, 0 if ctx.decode_only else 1, _stream()),
         "mingru_scan")
+    return out
+
+
+# ---------------------------------------------------------------------------
+# q and k normed over all heads, pairs (d, d + half) (csrc/joint_norm.cu); a real-gated linear recurrent unit (csrc/block_gates.cu)
+# ---------------------------------------------------------------------------
+def joint_norm_half_store(qkv: torch.Tensor, nq: int, nkv: int, hd: int, qk_dim: int, *, bias: Optional[torch.Tensor],
+                          q_norm_w: torch.Tensor, k_norm_w: torch.Tensor, eps: float, cos: Optional[torch.Tensor],
+                          sin: Optional[torch.Tensor], positions: torch.Tensor, slots: torch.Tensor, k_cache: torch.Tensor,
+                          v_cache: torch.Tensor, page_stride: int, page_size: int) -> None:
+    """Rows [q | k | v] of a fused projection, heads of ``hd`` numbers of which the first ``qk_dim`` count: add ``bias`` (float32
+    [columns]), norm q, and k, over all their heads together (float32 weights [heads * hd]), turn the first 2 * cos.shape[1]
+    numbers of q and k heads in the pairs (d, d + half); q back in place, k and v to the rows' page slots."""
+    _cuda(qkv, bias, q_norm_w, k_norm_w, cos, sin, positions, slots, k_cache, v_cache)
+    _i32(positions, "joint_norm_half_store positions")
+    _i32(slots, "joint_norm_half_store slots")
+    cols = (nq + 2 * nkv) * hd
+    if qkv.stride(1) != 1 or qkv.shape[1] < cols:
+        raise KernelError(f"joint_norm_half_store: rows of {qkv.shape[1]} numbers for {cols} columns")
+    for w, n in ((q_norm_w, nq * hd), (k_norm_w, nkv * hd), (bias, cols)):
+        if w is not None and (w.dtype != torch.float32 or w.numel() != n or not w.is_contiguous()):
+            raise KernelError(f"joint_norm_half_store: a weight or bias of {w.numel()} numbers, {n} float32 wanted")
+    if cos is not None and (cos.dtype != torch.float32 or sin is None or sin.shape != cos.shape or not (cos.is_contiguous() and sin.is_contiguous())):
+        raise KernelError("joint_norm_half_store: cos / sin must be contiguous float32 tables of one shape")
+    if k_cache.dtype != qkv.dtype or v_cache.dtype != qkv.dtype or positions.numel() != qkv.shape[0] or slots.numel() != qkv.shape[0]:
+        raise KernelError("joint_norm_half_store: the cache must have the rows' dtype, and every row a position and a slot")
+    _lib.check(_lib.load().oi_joint_norm_half_store(
+        qkv.data_ptr(), _code(qkv, "joint_norm_half_store"), qkv.stride(0), qkv.shape[0], nq, nkv, hd, qk_dim, _ptr(bias),
+        q_norm_w.data_ptr(), k_norm_w.data_ptr(), float(eps), _ptr(cos), _ptr(sin), 0 if cos is None else cos.shape[1],
+        0 if cos is None else cos.shape[0], positions.data_ptr(), slots.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
+        int(page_stride), int(page_size), _stream()), "joint_norm_half_store")
+
+
+def rglru_scan(out: torch.Tensor, u: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, rate: torch.Tensor, y: torch.Tensor,
+               y_bias: torch.Tensor, state: torch.Tensor, ctx) -> torch.Tensor:
+    """The rows of a step through a real-gated linear recurrent unit: ``u`` float32 [tokens, channels] behind its filter; ``w`` [2,
+    blocks, size, size] the two gates' matrices per part (out's type), ``bias`` float32 [2, channels]; ``rate`` float32 [channels],
+    the factor of -r in log a; out = S * gelu_tanh(y + y_bias) with ``y`` float32 rows; ``state`` float32 [slots, channels], read and
+    left behind. Two launches: the gates (which end the single rows) and, where a request brings several rows, the scan."""
+    _cuda(out, u, w, bias, rate, y, y_bias, state)
+    tokens, C = out.shape
+    _, blocks, size, _ = w.shape
+    if w.shape != (2, blocks, size, size) or blocks * size != C or not w.is_contiguous() or w.dtype not in (torch.float32, out.dtype):
+        raise KernelError(f"rglru_scan: the gates' matrices {tuple(w.shape)} {w.dtype} do not fit {C} channels of {out.dtype}")
+    for t, n in ((bias, 2 * C), (rate, C), (y_bias, C)):
+        if t.dtype != torch.float32 or t.numel() != n or not t.is_contiguous():
+            raise KernelError("rglru_scan: biases and rates must be contiguous float32 of the channels' number")
+    if u.dtype != torch.float32 or y.dtype != torch.float32 or u.shape != (tokens, C) or y.shape[0] != tokens or y.shape[1] < C \
+            or u.stride(1) != 1 or y.stride(1) != 1 or out.stride(1) != 1 or state.dtype != torch.float32 or state.shape[-1] != C \
+            or not state.is_contiguous():
+        raise KernelError(f"rglru_scan: u={tuple(u.shape)} y={tuple(y.shape)} out={tuple(out.shape)} state={tuple(state.shape)}")
+    step = (C + 3) & ~3
+    ab = torch.empty((tokens, 2 * step), dtype=torch.float32, device=out.device)
+    L = _lib.load()
+    meta = (ctx.cu_seqlens.data_ptr(), ctx.token_req.data_ptr(), ctx.state_slots.data_ptr())
+    code = _code(out, "rglru_scan")
+    _lib.check(L.oi_rglru_gates(u.data_ptr(), u.stride(0), w.data_ptr(), _code(w, "rglru_scan"), bias.data_ptr(), rate.data_ptr(),
+                                ab.data_ptr(), ab.stride(0), step, y.data_ptr(), y.stride(0), y_bias.data_ptr(), out.data_ptr(), code,
+                                out.stride(0), state.data_ptr(), state.stride(0), *meta, tokens, blocks, size, _stream()), "rglru_gates")
+    if not ctx.decode_only:
+        _lib.check(L.oi_affine_scan(out.data_ptr(), code, out.stride(0), ab.data_ptr(), ab.stride(0), step, y.data_ptr(), y.stride(0),
+                                    y_bias.data_ptr(), state.data_ptr(), state.stride(0), *meta, tokens, ctx.num_requests, C,
+                                    _stream()), "affine_scan")
     return out

@@ -1,2 +1,2 @@
 """Built-in architectures. Importing this package registers them."""
-from . import bubalix, delunex, linurax, luzitar, pilonex, qwen3  # noqa: F401
+from . import bubalix, delunex, linurax, luzitar, pilonex, qwen3, rolevik  # noqa: F401

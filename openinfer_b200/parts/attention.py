@@ -24,6 +24,8 @@ Also from the spec: biases on q, k and v; a unit norm of q and k heads AFTER the
 numbers, no weight) instead of the weighted norm before it; with a window, a number of first keys of the sequence that stay
 visible behind it (their pages are kept). A layer with biases or the norm behind the rotation prepares its rows with one
 kernel of its own (csrc/sandwich_ops.cu: bias, rotation, norm, cache write) and hands the attention kernels ready queries.
+``joint_norm_eps``: q, and k, normed over all their heads together (csrc/joint_norm.cu: bias, norm, rotation of the pairs
+(d, d + half), cache write). ``chunked``: ``window`` is the size of chunks counted from position 0, a query sees its own chunk.
 A bias in front of the filter is carried behind it: filter(u + b)_t = filter(u)_t + b * (sum of the taps that fall on
 positions >= 0), a small table by position that the same kernel adds.
 """
@@ -70,15 +72,23 @@ class Attention(Mixer):
         self.qkv_cols = self.q_dim + 2 * self.kv_dim
         self.gate_off = self.qkv_cols                      # the gate's columns of the fused projection, behind q | k | v
         self.in_cols = -(-(self.qkv_cols + (s.num_heads if s.head_gate else 0)) // 8) * 8
+        if s.chunked and s.keep_first:
+            raise ValueError("attention: chunks keep no first keys")
+        # the mask as the kernels take it: 0 every key, > 0 a window, < 0 chunks of that size
+        self.mask = (-int(s.window) if s.chunked else int(s.window)) if s.window else 0
         if s.keep_first < 0 or s.unit_norm_after_rotation_eps < 0.0:
             raise ValueError("attention: keep_first and the unit norm's eps cannot be negative")
         if s.unit_norm_after_rotation_eps > 0.0 and s.qk_norm is not None:
             raise ValueError("attention: q and k are normed before the rotation or behind it, not both")
         self.keep_first = int(s.keep_first) if s.window else 0
-        # rows prepared by rope_norm_store (bias, rotation, unit norm, cache write) instead of the norm-then-rotate kernel
-        self.own_prepare = bool(s.qkv_bias or s.unit_norm_after_rotation_eps > 0.0)
+        self.joint_norm = s.joint_norm_eps > 0.0
+        if self.joint_norm and (s.qk_norm is not None or s.unit_norm_after_rotation_eps > 0.0 or s.conv_taps > 0):
+            raise ValueError("attention: a norm over all heads together goes with no other norm and no filter")
+        # rows prepared by rope_norm_store (bias, rotation, unit norm, cache write) or joint_norm_half_store (bias, norm over
+        # all heads, rotation, cache write) instead of the norm-then-rotate kernel
+        self.own_prepare = bool(s.qkv_bias or s.unit_norm_after_rotation_eps > 0.0 or self.joint_norm)
         if self.own_prepare and s.position.kind != "none" and getattr(s.position, "interleaved", False):
-            raise ValueError("attention: the rotation in front of a unit norm turns the pairs (d, d + half)")
+            raise ValueError("attention: a layer that prepares its rows with a kernel of its own turns the pairs (d, d + half)")
         self.bias_tab: Optional[torch.Tensor] = None
         self.has_mods = bool(s.sink or s.score_cap > 0.0 or s.distance_slope_exponent > 0.0 or s.q_temperature is not None
                              or self.keep_first > 0)
@@ -94,7 +104,7 @@ class Attention(Mixer):
 
     def kv_need(self) -> Optional[KvNeed]:
         s = self.spec
-        return KvNeed(s.num_kv_heads, s.head_dim, s.window, keep_first=self.keep_first)
+        return KvNeed(s.num_kv_heads, s.head_dim, s.window, chunked=bool(s.chunked and s.window), keep_first=self.keep_first)
 
     def state_needs(self):
         s = self.spec
@@ -112,6 +122,9 @@ class Attention(Mixer):
         if s.qk_norm is not None:
             p[s.q_norm_name] = ParamInfo((self.qk,), ("one_plus_normal", 0.02))
             p[s.k_norm_name] = ParamInfo((self.qk,), ("one_plus_normal", 0.02))
+        if self.joint_norm:
+            p[s.q_norm_name] = ParamInfo((s.num_heads * self.qk,), ("one_plus_normal", 0.1))
+            p[s.k_norm_name] = ParamInfo((s.num_kv_heads * self.qk,), ("one_plus_normal", 0.1))
         if s.conv_taps > 0:
             for name, rows in ((s.q_name, s.num_heads * self.qk), (s.k_name, s.num_kv_heads * self.qk), (s.v_name, s.num_kv_heads * self.vd)):
                 p[name + s.conv_suffix] = ParamInfo((rows, s.conv_taps), ("normal_around", 0.2, 1.0 / s.conv_taps))
@@ -169,6 +182,10 @@ class Attention(Mixer):
             wide[:, :, : self.vd] = o.view(o.shape[0], s.num_heads, self.vd)
             o = wide.view(o.shape[0], s.num_heads * hd)
         self.w_o = o.contiguous()
+        if self.joint_norm:
+            self.q_norm_w, self.k_norm_w = (
+                rows_padded(tensors[n].to(torch.float32)[:, None], heads, self.qk)[:, 0].contiguous()
+                for n, heads in ((s.q_norm_name, s.num_heads), (s.k_norm_name, s.num_kv_heads)))
         if self.spec.qk_norm is not None:
             def norm_padded(w):
                 if self.qk == hd:
@@ -219,17 +236,27 @@ class Attention(Mixer):
         cos, sin = self.tables if self.tables is not None else (None, None)
         qn = s.qk_norm
         out = torch.empty((x.shape[0], self.q_dim), dtype=x.dtype, device=x.device)
-        if self.own_prepare:
+        if self.joint_norm:
+            # bias, norm over all heads, rotation and cache write in one kernel
+            if not binding.owns_kv:
+                raise RuntimeError("attention: a layer with a norm over all heads owns its cache")
+            ops.joint_norm_half_store(qkv, s.num_heads, s.num_kv_heads, s.head_dim, self.qk,
+                                      bias=None if self.bias_tab is None else self.bias_tab[0], q_norm_w=self.q_norm_w,
+                                      k_norm_w=self.k_norm_w, eps=s.joint_norm_eps, cos=cos, sin=sin, positions=ctx.positions,
+                                      slots=group.slot_mapping, k_cache=k_cache, v_cache=v_cache, page_stride=page_stride,
+                                      page_size=ctx.cache.page_size)
+        elif self.own_prepare:
             # bias, rotation, unit norm and cache write in one kernel of the layer's own; the attention kernels get ready rows
             ops.rope_norm_store(qkv, s.num_heads, s.num_kv_heads, s.head_dim, self.qk, bias_tab=self.bias_tab, cos=cos, sin=sin,
                                 unit_norm=s.unit_norm_after_rotation_eps > 0.0, eps=s.unit_norm_after_rotation_eps,
                                 positions=ctx.positions, slots=group.slot_mapping if binding.owns_kv else None,
                                 k_cache=k_cache if binding.owns_kv else None, v_cache=v_cache if binding.owns_kv else None,
                                 page_stride=page_stride, page_size=ctx.cache.page_size, write_kv=binding.owns_kv)
+        if self.own_prepare:
             step = attn_kernels.attention_step(ctx, group, qkv, out, k_cache, page_stride, s.num_heads, s.num_kv_heads,
-                                               s.head_dim, s.window, mods=self.has_mods, keep_first=self.keep_first)
+                                               s.head_dim, self.mask, mods=self.has_mods, keep_first=self.keep_first)
             layer = attn_kernels.attention_layer(qkv, out, k_cache, v_cache, s.num_heads, s.num_kv_heads, s.head_dim, self.scale,
-                                                 s.window, write_kv=False, rope_mode=0, mods=self.mods)
+                                                 self.mask, write_kv=False, rope_mode=0, mods=self.mods)
             attn_kernels.run_attention(step, layer)
             if s.head_gate:
                 ops.head_gate(out, raw[:, self.gate_off: self.gate_off + s.num_heads], s.num_heads, s.head_dim)
@@ -237,10 +264,10 @@ class Attention(Mixer):
         # One native call: the norm + rotation + cache write (in a kernel of its own, or inside the decode kernel when
         # the step is single tokens in one wave), then the attention kernel(s) that take the step's shape.
         step = attn_kernels.attention_step(ctx, group, qkv, out, k_cache, page_stride, s.num_heads, s.num_kv_heads,
-                                           s.head_dim, s.window, cos=cos, q_norm_w=self.q_norm_w, mods=self.has_mods,
+                                           s.head_dim, self.mask, cos=cos, q_norm_w=self.q_norm_w, mods=self.has_mods,
                                            keep_first=self.keep_first)
         layer = attn_kernels.attention_layer(
-            qkv, out, k_cache, v_cache, s.num_heads, s.num_kv_heads, s.head_dim, self.scale, s.window,
+            qkv, out, k_cache, v_cache, s.num_heads, s.num_kv_heads, s.head_dim, self.scale, self.mask,
             q_norm_w=self.q_norm_w, k_norm_w=self.k_norm_w, eps=qn.eps * self.norm_eps_factor if qn else 0.0,
             weight_offset=qn.weight_offset if qn else 0.0, cos=cos, sin=sin, write_kv=binding.owns_kv, rope_mode=1,
             interleaved=bool(getattr(s.position, "interleaved", False)), mods=self.mods)

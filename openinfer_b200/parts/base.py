@@ -104,6 +104,9 @@ class Block(Part):
                 binding: CacheBinding) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
         raise NotImplementedError
 
+    def loaded(self) -> None:
+        """Called once when all of the block's parts hold their tensors: for what is formed from several parts' tensors."""
+
     def sub_parts(self) -> Dict[str, Part]:
         """Tensor-name prefix (relative to the block's own name) -> part."""
         return {}

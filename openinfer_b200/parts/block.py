@@ -11,7 +11,7 @@ import torch
 
 from ..kernels import ops
 from .base import Block, CacheBinding, Part
-from .norm import RmsNorm
+from .norm import LayerNorm, RmsNorm
 from .registry import build_feed_forward, build_mixer, build_norm, build_stream_part, register_block
 from .spec import BlockSpec
 
@@ -57,7 +57,9 @@ class BranchNormBlock(Block):
     The stream is float32 whatever the model's type: the branches get it rounded to the model's type (by the filter, or
     by the kernel that ends the branch before), return float32, and one kernel norms a branch's output, adds it, and,
     after the block's last branch, forms the average. ``spec.input_norm`` is the norm of the mixer's output,
-    ``spec.post_norm`` that of the feed-forward's.
+    ``spec.post_norm`` that of the feed-forward's; either may be a layer norm. With ``mixer_scale`` / ``feed_forward_scale``
+    the normed branch is multiplied by a weight per channel (which is multiplied into the norm's weight once). A mixer of
+    two sides whose results are normed first hands both over, and the same kernel forms their sum.
     """
 
     def __init__(self, spec: BlockSpec) -> None:
@@ -69,8 +71,24 @@ class BranchNormBlock(Block):
         self.conv = build_stream_part(spec.input_conv) if spec.input_conv is not None else None
         self.depth = build_stream_part(spec.depth_average) if spec.depth_average is not None else None
         for n in (self.mixer_norm, self.ff_norm):
-            if n is not None and not isinstance(n, RmsNorm):
-                raise ValueError("a branchnorm block needs rms norms")
+            if n is not None and not isinstance(n, (RmsNorm, LayerNorm)):
+                raise ValueError("a branchnorm block needs rms or layer norms")
+        self.mixer_scale = build_stream_part(spec.mixer_scale) if spec.mixer_scale is not None else None
+        self.ff_scale = (build_stream_part(spec.feed_forward_scale)
+                         if spec.feed_forward_scale is not None and self.feed_forward is not None else None)
+        # branches that join by the general kernel (ops.branch_join): layer norms, scaled branches, normed pairs
+        self.general_join = bool(self.mixer_scale is not None or self.ff_scale is not None or getattr(self._mixer, "returns_normed_pair", False)
+                                 or any(isinstance(n, LayerNorm) for n in (self.mixer_norm, self.ff_norm)))
+        if self.general_join and self.depth is not None:
+            raise ValueError("a branchnorm block averages over depth with plain rms norms only")
+        self._join_weights: Dict[int, torch.Tensor] = {}
+
+    def loaded(self) -> None:
+        if self.general_join:      # (weight_offset + weight) * scale in float32, formed once
+            for norm, scale in ((self.mixer_norm, self.mixer_scale), (self.ff_norm, self.ff_scale)):
+                if norm is not None:
+                    w = norm.weight.to(torch.float32) + norm.spec.weight_offset
+                    self._join_weights[id(norm)] = (w * scale.weight.to(torch.float32) if scale is not None else w).contiguous()
 
     wants_history = property(lambda self: self.depth is not None)
     stream_dtype = torch.float32
@@ -89,6 +107,10 @@ class BranchNormBlock(Block):
             parts[s.input_conv_name] = self.conv
         if self.depth is not None:
             parts[s.depth_average_name] = self.depth
+        if self.mixer_scale is not None:
+            parts[s.mixer_scale_name] = self.mixer_scale
+        if self.ff_scale is not None:
+            parts[s.feed_forward_scale_name] = self.ff_scale
         return parts
 
     def state_needs(self):
@@ -108,12 +130,16 @@ class BranchNormBlock(Block):
                 u = h if dtype == torch.float32 else h.to(dtype)
         ctx.scratch.pop("stream_low", None)
         wide = {"out_dtype": torch.float32}      # parts that can, hand their branch back unrounded
+        pair = {"as_normed_pair": True} if getattr(self._mixer, "returns_normed_pair", False) else {}
         a = self._mixer.forward(u, ctx, dataclasses.replace(binding, states=binding.states[n_conv:]),
-                                **(wide if getattr(self._mixer, "takes_out_dtype", False) else {}))
+                                **(wide if getattr(self._mixer, "takes_out_dtype", False) else {}), **pair)
         hist = ctx.scratch.get("stream_history") if self.depth is not None else None
         low = torch.empty(h.shape, dtype=dtype, device=h.device) if dtype != torch.float32 else None
 
         def join(branch, norm, last, low_out):
+            if self.general_join:
+                ops.branch_join(h, branch, weight=self._join_weights[id(norm)], center=isinstance(norm, LayerNorm), eps=norm.spec.eps, low=low_out)
+                return
             kw = {}
             if last and hist is not None:
                 kw = dict(history=hist[0], n_prev=hist[1], coef=self.depth.weight)

@@ -15,7 +15,7 @@ from ..kernels import attention as attn_kernels
 from ..kernels import lib as _lib
 from ..kernels import native, ops
 from ..kernels.linear import ensure_library, linear
-from .base import Block, CacheBinding
+from .base import Block, CacheBinding, Part
 from .registry import build_block, build_norm
 from .spec import LayerCall, ModelSpec, ParamInfo
 
@@ -85,6 +85,7 @@ class Model:
                 full = bspec.name + prefix
                 part.load({local: tensors[self._tensor_name(full, local)] for local in part.parameters()})
                 part.prepare(self.device, self.dtype)
+            block.loaded()
         self.final_norm.load({local: tensors[s.final_norm_name + local] for local in self.final_norm.parameters()})
         if self.embedding_norm is not None:
             self.embedding_norm.load({local: tensors[s.embedding_norm_name + local] for local in self.embedding_norm.parameters()})
@@ -100,12 +101,17 @@ class Model:
                 seen.add(t.data_ptr())
                 total += t.numel() * t.element_size()
 
+        def add_part(part):
+            for v in vars(part).values():
+                if isinstance(v, torch.Tensor):
+                    add(v)
+                elif isinstance(v, Part):        # parts made of parts (two mixers side by side, a shared expert)
+                    add_part(v)
+
         add(self.head)
         for block in self.blocks:
             for part in block.sub_parts().values():
-                for v in vars(part).values():
-                    if isinstance(v, torch.Tensor):
-                        add(v)
+                add_part(part)
         add(getattr(self.final_norm, "weight", None))
         return total
 
@@ -124,7 +130,9 @@ class Model:
                 needs[i] = need
             elif need is not None and needs.get(c.read_cache_of) is not None:
                 src = needs[c.read_cache_of]
-                if src.window is not None and (need.window is None or need.window > src.window):
+                if src.window is not None and (need.chunked or src.chunked) and (need.window, need.chunked) != (src.window, src.chunked):
+                    needs[c.read_cache_of] = _dc.replace(src, window=None, chunked=False)     # readers of other chunks: keep every page
+                elif src.window is not None and (need.window is None or need.window > src.window):
                     needs[c.read_cache_of] = _dc.replace(src, window=need.window)
         self.bindings = []
         for i, c in enumerate(self.calls):
@@ -217,7 +225,7 @@ class Model:
             self._native = self._native_description_branch(ctx)
             return self._native
         if not own(self.final_norm, RmsNorm) or not all(
-                own(b, PreNormBlock) and own(b.mixer, Attention) and own(b.feed_forward, GatedMlp)
+                own(b, PreNormBlock) and own(b.mixer, Attention) and not b.mixer.joint_norm and own(b.feed_forward, GatedMlp)
                 and own(b.input_norm, RmsNorm) and own(b.post_norm, RmsNorm) for b in self.blocks):
             return None
         codes = native.DTYPE_CODE
@@ -231,7 +239,7 @@ class Model:
             k_cache, v_cache, page_stride = cache.kv_views(binding.kv)
             qkv_rows = at.q_dim + 2 * at.kv_dim if binding.owns_kv else at.q_dim
             cos, sin = at.tables if at.tables is not None else (None, None)
-            key = (binding.kv.group, s.num_heads, s.num_kv_heads, s.head_dim, s.window, qkv_rows, cos is not None,
+            key = (binding.kv.group, s.num_heads, s.num_kv_heads, s.head_dim, at.mask, qkv_rows, cos is not None,
                    None if at.q_norm_w is None else at.q_norm_w.dtype)
             if key not in keys:
                 keys.append(key)
@@ -255,7 +263,7 @@ class Model:
             a.norm_dtype = 0 if at.q_norm_w is None else codes[at.q_norm_w.dtype]
             a.cos_tab, a.sin_tab = (0, 0) if cos is None else (cos.data_ptr(), sin.data_ptr())
             a.rot_half, a.max_pos = (0, 0) if cos is None else (cos.shape[1], cos.shape[0])
-            a.nq, a.nkv, a.hd, a.window = s.num_heads, s.num_kv_heads, s.head_dim, int(s.window) if s.window else 0
+            a.nq, a.nkv, a.hd, a.window = s.num_heads, s.num_kv_heads, s.head_dim, at.mask
             a.scale, a.eps, a.w_offset = at.scale, (qn.eps * at.norm_eps_factor if qn else 0.0), (qn.weight_offset if qn else 0.0)
             a.write_kv, a.rope_mode = (1 if binding.owns_kv else 0), 1
             a.interleaved = 1 if getattr(s.position, "interleaved", False) else 0
@@ -285,7 +293,7 @@ class Model:
             return type(obj) is cls
 
         for i, b in enumerate(self.blocks):
-            ok = (own(b.mixer, LatentAttention) and b.mixer.spec.absorb == "weights" and own(b.mixer_norm, RmsNorm)
+            ok = (not b.general_join and own(b.mixer, LatentAttention) and b.mixer.spec.absorb == "weights" and own(b.mixer_norm, RmsNorm)
                   and (b.feed_forward is None or (own(b.feed_forward, DenseMlp) and own(b.ff_norm, RmsNorm)))
                   and (b.conv is None or own(b.conv, ShortConv)) and (b.depth is None or own(b.depth, DepthAverage)))
             if not ok or (b.conv is None and self.dtype != torch.float32 and i == 0):
@@ -415,7 +423,7 @@ class Model:
             cos = at.tables[0] if at.tables is not None else None
             s = attn_kernels.attention_step(ctx, ctx.groups[binding.kv.group], qkv.view(-1)[: T * L.qkv_rows].view(T, L.qkv_rows),
                                             attn.view(-1)[: T * at.q_dim].view(T, at.q_dim), k_cache, page_stride,
-                                            L.attn.nq, L.attn.nkv, L.attn.hd, at.spec.window, cos=cos, q_norm_w=at.q_norm_w)
+                                            L.attn.nq, L.attn.nkv, L.attn.hd, at.mask, cos=cos, q_norm_w=at.q_norm_w)
             kept.append(s)
             ctypes.memmove(ctypes.byref(steps[j]), ctypes.byref(s), ctypes.sizeof(native.AttnStep))
         xs = ssq = None

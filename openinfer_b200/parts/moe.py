@@ -10,6 +10,10 @@ choices in a fixed order (csrc/moe.cu). Nothing of a step's routing is read on t
 ``keep_groups`` of ``groups`` equal groups of neighbours (a group's score: the sum of its two largest choice scores); the
 weights are the chosen experts' s (without the correction) divided by their sum.
 
+``routing`` "softmax_groups": the same choice with s the softmax over all rows of the router and a group's score its largest choice
+score; the weights are the chosen s times ``weight_scale``. With ``identity`` the router (and the correction and the groups) has
+that many rows behind the experts': choosing one of them adds the input itself, times its weight.
+
 ``routing`` "table": there is no router; an integer table [vocab, top] gives every token id its experts (the entries of a
 row differ), each weighted 1 / top. ``shared``: one more expert of the same form that every row uses; its result (float32)
 is added by the kernel that sums a row's choices.
@@ -33,14 +37,18 @@ class RoutedExperts(FeedForward):
     def __init__(self, spec: RoutedExpertsSpec) -> None:
         super().__init__(spec)
         s = spec
-        if not 0 < s.top <= s.experts or s.top > 32 or s.intermediate_size <= 0:
+        if not 0 < s.top <= s.experts + s.identity or s.experts <= 0 or s.top > 32 or s.intermediate_size <= 0:
             raise ValueError(f"routed_experts: {s.top} of {s.experts} experts (at most 32 a row), ff {s.intermediate_size}")
         ops.glu_code(s.activation)          # refuses a name no kernel knows
-        if s.routing not in ("softmax_top", "table", "sigmoid_groups"):
-            raise ValueError(f"routed_experts: routing must be 'softmax_top', 'sigmoid_groups' or 'table', got {s.routing!r}")
-        if s.routing == "sigmoid_groups" and (s.groups < 1 or not 1 <= s.keep_groups <= s.groups or s.experts % s.groups
-                                              or (s.experts // s.groups) * s.keep_groups < s.top):
-            raise ValueError(f"routed_experts: {s.experts} experts in {s.groups} groups of which {s.keep_groups} are kept "
+        if s.routing not in ("softmax_top", "table", "sigmoid_groups", "softmax_groups"):
+            raise ValueError(f"routed_experts: routing must be 'softmax_top', 'sigmoid_groups', 'softmax_groups' or 'table', got {s.routing!r}")
+        self.grouped = s.routing in ("sigmoid_groups", "softmax_groups")
+        if s.identity < 0 or (s.identity and s.routing != "softmax_groups"):
+            raise ValueError("routed_experts: choices that stand for the input go with 'softmax_groups' routing")
+        self.choices = s.experts + s.identity
+        if self.grouped and (s.groups < 1 or not 1 <= s.keep_groups <= s.groups or self.choices % s.groups
+                             or (self.choices // s.groups) * s.keep_groups < s.top):
+            raise ValueError(f"routed_experts: {self.choices} choices in {s.groups} groups of which {s.keep_groups} are kept "
                              f"cannot give {s.top} choices")
         if s.routing == "table" and s.vocab_size <= 0:
             raise ValueError("routed_experts: routing by a table needs the vocabulary's size")
@@ -63,9 +71,9 @@ class RoutedExperts(FeedForward):
         if s.routing == "table":
             p = {s.table_name: ParamInfo((s.vocab_size, s.top), ("distinct_below", s.experts), integer=True)}
         else:
-            p = {s.router_name: ParamInfo((s.experts, W), ("normal", W ** -0.5))}
-            if s.routing == "sigmoid_groups":
-                p[s.correction_name] = ParamInfo((s.experts,), ("normal", 0.1))
+            p = {s.router_name: ParamInfo((self.choices, W), ("normal", W ** -0.5))}
+            if self.grouped:
+                p[s.correction_name] = ParamInfo((self.choices,), ("normal", 0.1))
         for e in range(s.experts):
             g, u, d = self._names(e)
             p[g] = ParamInfo((F, W), ("normal", W ** -0.5))
@@ -82,7 +90,7 @@ class RoutedExperts(FeedForward):
             self.table = tensors[s.table_name].to(torch.int32).contiguous()
         else:
             self.w_router = tensors[s.router_name].contiguous()
-            if s.routing == "sigmoid_groups":
+            if self.grouped:
                 self.correction = tensors[s.correction_name].to(torch.float32).contiguous()
         if self.shared is not None:
             self.shared.load({local: tensors[s.shared_name + local] for local in self.shared.parameters()})
@@ -96,9 +104,9 @@ class RoutedExperts(FeedForward):
             x = x.contiguous()
         if s.routing == "table":
             routing = ops.moe_route_table(ctx.token_ids, self.table, s.experts)
-        elif s.routing == "sigmoid_groups":
-            routing = ops.moe_route(x, self.w_router, s.top, scoring="sigmoid_groups", correction=self.correction, groups=s.groups,
-                                    keep_groups=s.keep_groups)
+        elif self.grouped:
+            routing = ops.moe_route(x, self.w_router, s.top, scoring=s.routing, correction=self.correction, groups=s.groups,
+                                    keep_groups=s.keep_groups, identity=s.identity, weight_scale=s.weight_scale)
         else:
             routing = ops.moe_route(x, self.w_router, s.top)
         add = self.shared.forward(x, ctx, out_dtype=torch.float32) if self.shared is not None else None

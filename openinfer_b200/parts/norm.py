@@ -41,6 +41,30 @@ class RmsNorm(Norm):
                            weight_offset=self.spec.weight_offset)
 
 
+@register_norm("layer")
+class LayerNorm(Norm):
+    """A layer norm without a bias: out = (x - mean) / sqrt(mean((x - mean)^2) + eps) * (weight_offset + weight), float32
+    arithmetic. Blocks that fuse it with the residual add read ``weight``."""
+
+    def __init__(self, spec: NormSpec) -> None:
+        super().__init__(spec)
+        self.weight: Optional[torch.Tensor] = None
+
+    def parameters(self) -> Dict[str, ParamInfo]:
+        return {self.spec.param_name: ParamInfo((self.spec.size,), ("one_plus_normal", 0.1))}
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.weight = tensors[self.spec.param_name].contiguous()
+
+    def __call__(self, x: torch.Tensor, *, delta: Optional[torch.Tensor] = None, row_idx: Optional[torch.Tensor] = None,
+                 out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+        if delta is not None:
+            raise ValueError("a layer norm takes no pending branch")
+        rows = x.shape[0] if row_idx is None else row_idx.numel()
+        out = torch.empty((rows, x.shape[1]), dtype=out_dtype or x.dtype, device=x.device)
+        return ops.rmsnorm_cast(out, x, self.weight, self.spec.eps, row_idx=row_idx, weight_offset=self.spec.weight_offset, center=True)
+
+
 @register_norm("dyt")
 class DynamicTanh(Norm):
     """Dynamic Tanh: out = tanh(alpha * x) * w + b with a learned scalar alpha; no mean and no variance are formed

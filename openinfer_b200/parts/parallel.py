@@ -1,14 +1,16 @@
-"""Two mixers side by side: both read the same rows, the result is left_scale * left + right_scale * right.
+"""Two mixers side by side: both read the same rows, the result is left_scale * left + right_scale * right, the two results
+RMS-normed over the width first when the spec says so (``out_norm_eps``).
 
 The two are whatever mixers their specs name (an attention beside a recurrence, for instance); each keeps its own tensors
 under its own prefix, the cache entry is the one that asks for pages, and the state slots are the left's followed by the
 right's. Both hand their results back in float32; the weighted sum is formed by the kernel that carries a block's result into
-its streams when the block asks for the pair (``as_pair``), else by a kernel of its own.
+its streams when the block asks for the pair (``as_pair``; ``as_normed_pair`` where the results are normed), else by a kernel of its
+own.
 """
 from __future__ import annotations
 
 import dataclasses
-from typing import Dict, List, Optional
+from typing import Dict, List, Optional, Tuple
 
 import torch
 
@@ -22,7 +24,6 @@ from .spec import ParallelMixerSpec, ParamInfo
 @register_mixer("parallel")
 class ParallelMixer(Mixer):
     takes_out_dtype = True
-    returns_pair = True      # forward(as_pair=True) hands back both sides and their scales instead of the sum
 
     def __init__(self, spec: ParallelMixerSpec) -> None:
         super().__init__(spec)
@@ -33,6 +34,13 @@ class ParallelMixer(Mixer):
         for side in (self.left, self.right):
             if not getattr(side, "takes_out_dtype", False):
                 raise ValueError(f"a parallel mixer needs sides that can return float32, {type(side).__name__} cannot")
+        self.normed = spec.out_norm_eps > 0.0
+        self.out_norms: Optional[Tuple[torch.Tensor, torch.Tensor]] = None       # float32 weights, left and right
+
+    # forward(as_pair=True) hands back both sides and their scales instead of the sum; forward(as_normed_pair=True) a
+    # ``NormedPair``, where the sum is one of normed sides
+    returns_pair = property(lambda self: not self.normed)
+    returns_normed_pair = property(lambda self: self.normed)
 
     @property
     def graph_safe(self) -> bool:
@@ -42,11 +50,17 @@ class ParallelMixer(Mixer):
         return ((self.spec.left_name, self.left), (self.spec.right_name, self.right))
 
     def parameters(self) -> Dict[str, ParamInfo]:
-        return {prefix + name: info for prefix, side in self._sides() for name, info in side.parameters().items()}
+        p = {prefix + name: info for prefix, side in self._sides() for name, info in side.parameters().items()}
+        if self.normed:
+            for prefix, side in self._sides():
+                p[prefix + self.spec.out_norm_name] = ParamInfo((side.spec.hidden_size,), ("one_plus_normal", 0.1))
+        return p
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         for prefix, side in self._sides():
             side.load({name: tensors[prefix + name] for name in side.parameters()})
+        if self.normed:
+            self.out_norms = tuple(tensors[prefix + self.spec.out_norm_name].to(torch.float32).contiguous() for prefix, _ in self._sides())
 
     def prepare(self, device: torch.device, dtype: torch.dtype) -> None:
         self.left.prepare(device, dtype)
@@ -58,14 +72,21 @@ class ParallelMixer(Mixer):
     def state_needs(self) -> List[StateNeed]:
         return self.left.state_needs() + self.right.state_needs()
 
-    def forward(self, x: torch.Tensor, ctx, binding: CacheBinding, out_dtype: Optional[torch.dtype] = None, as_pair: bool = False):
+    def forward(self, x: torch.Tensor, ctx, binding: CacheBinding, out_dtype: Optional[torch.dtype] = None, as_pair: bool = False,
+                as_normed_pair: bool = False):
         n_left = len(self.left.state_needs())
         kv_left = self.left.kv_need() is not None
         lb = dataclasses.replace(binding, kv=binding.kv if kv_left else None, states=binding.states[:n_left])
         rb = dataclasses.replace(binding, kv=None if kv_left else binding.kv, states=binding.states[n_left:])
         a = self.left.forward(x, ctx, lb, out_dtype=torch.float32)
         b = self.right.forward(x, ctx, rb, out_dtype=torch.float32)
-        if as_pair:
+        if self.normed:
+            pair = ops.NormedPair(a, b, *self.out_norms, float(self.spec.left_scale), float(self.spec.right_scale), self.spec.out_norm_eps)
+            if as_normed_pair:
+                return pair
+            out = ops.branch_join(None, pair, out=torch.empty_like(a))
+        elif as_pair:
             return a, b, float(self.spec.left_scale), float(self.spec.right_scale)
-        out = ops.scaled_sum(torch.empty_like(a), a, b, self.spec.left_scale, self.spec.right_scale)
+        else:
+            out = ops.scaled_sum(torch.empty_like(a), a, b, self.spec.left_scale, self.spec.right_scale)
         return out if out_dtype in (None, torch.float32) else out.to(out_dtype)

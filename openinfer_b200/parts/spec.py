@@ -34,6 +34,7 @@ class NormSpec:
     eps: float = 1e-6
     weight_offset: float = 0.0  # scale is (weight_offset + w)
     param_name: str = "weight"  # local tensor name (appended to the prefix the enclosing part gives the norm)
+    # kind "layer" (a layer norm without a bias): the row's mean is taken off before the root mean square is formed
     # kind "dyt" (Dynamic Tanh: tanh(alpha x) w + b, no mean and no variance; eps is not used): the bias vector and the
     # scalar alpha are stored beside the weight under its name + these suffixes
     bias_suffix: str = ".b"
@@ -72,6 +73,7 @@ class AttentionSpec:
     position: PositionSpec = PositionSpec(kind="none")
     qk_norm: Optional[NormSpec] = None      # per-head norm over head_dim, before the rotation
     window: Optional[int] = None            # keys visible to a query, itself included; None = all
+    chunked: bool = False                   # ``window`` is the size of chunks counted from position 0: a query sees the keys of its own
     # queries / keys and values of other sizes than head_dim (None: head_dim). head_dim is then the cached row, a multiple
     # of 8 that holds both; the projections are padded with zero rows at load time and the norm's constants follow
     qk_dim: Optional[int] = None
@@ -101,6 +103,9 @@ class AttentionSpec:
     # > 0: AFTER the rotation q and k heads are divided by their root mean square over qk_dim numbers (no weight), with
     # this eps inside the root; takes the place of ``qk_norm``, which norms before the rotation
     unit_norm_after_rotation_eps: float = 0.0
+    # > 0: q, and k, are normed over ALL their heads together (one root mean square a row, weights ``q_norm_name`` [heads *
+    # qk_dim] and ``k_norm_name``) before the rotation, with this eps; takes the place of ``qk_norm``
+    joint_norm_eps: float = 0.0
     # with a window: the first ``keep_first`` keys of a sequence stay visible to every later query (at their true
     # positions), and their pages are never given back
     keep_first: int = 0
@@ -242,8 +247,11 @@ class RoutedExpertsSpec:
     # ``table_name`` [vocab_size, top] gives every token id its experts, each weighted 1 / top. "sigmoid_groups": scores
     # s = sigmoid(logit); the choice goes by s + a stored correction (``correction_name`` [experts]) among the experts of
     # the ``keep_groups`` best of ``groups`` equal groups of neighbours (a group's score: the sum of its two largest choice
-    # scores); the weights are the chosen experts' s divided by their sum
+    # scores); the weights are the chosen experts' s divided by their sum. "softmax_groups": s is the softmax over all rows of
+    # the router, a group's score its largest choice score, the weights the chosen s times ``weight_scale``
     routing: str = "softmax_top"
+    weight_scale: float = 1.0
+    identity: int = 0                       # rows of the router (and of correction and groups) behind the experts' that stand for the input itself
     correction_name: str = "correction"
     groups: int = 1
     keep_groups: int = 1
@@ -270,9 +278,11 @@ class MatrixMemorySpec:
 
 @dataclasses.dataclass(frozen=True)
 class GatedDeltaSpec:
-    """A recurrent mixer with a matrix C [qk_dim, v_dim] per head updated by the delta rule, one decay per head and key
-    channel; queries, keys and values pass a short causal filter over time and silu first. The decay and the output
-    gate come through low-rank products whose inner sizes the checkpoint decides."""
+    """A recurrent mixer with a matrix C [qk_dim, v_dim] per head updated by the delta rule; queries, keys and values pass a
+    short causal filter over time and silu first. ``decay_per`` "channel": one decay per head and key channel; the decay and
+    the output gate come through low-rank products (a2 a1, g2 g1) whose inner sizes the checkpoint decides. "head": one decay
+    per head (``a`` [heads, hidden]) and a full output gate (``g`` [heads * v_dim, hidden]). ``gate_activation``: what the
+    gate's raw value goes through, "sigmoid" or "silu"."""
 
     kind: str = "gated_delta"
     hidden_size: int = 0
@@ -284,6 +294,8 @@ class GatedDeltaSpec:
     eps: float = 1e-6
     decay_rank: int = 0                     # what random weights use; a checkpoint's own sizes win
     gate_rank: int = 0
+    decay_per: str = "channel"
+    gate_activation: str = "sigmoid"
 
 
 @dataclasses.dataclass(frozen=True)
@@ -355,8 +367,42 @@ class MinGruSpec:
 
 
 @dataclasses.dataclass(frozen=True)
+class RgLruSpec:
+    """A real-gated linear recurrent unit behind a short causal filter, beside a gate (Griffin's recurrent block): y = gelu_tanh(W_y
+    x + b), u = filter(W_x x + b) + b'; u in ``blocks`` equal parts, per part r = sigmoid(R u + b), i = sigmoid(I u + b); a = exp(-c r
+    softplus(lambda)), S_t = a S_(t-1) + sqrt(1 - a^2) i u, the result W_o (S * y). S and the filter's last taps - 1 inputs are
+    float32 state per request, zero at its start."""
+
+    kind: str = "rglru"
+    hidden_size: int = 0
+    channels: int = 0
+    blocks: int = 1
+    conv_taps: int = 1
+    rate: float = 8.0                       # c
+    y_name: str = "y"
+    x_name: str = "x"
+    conv_name: str = "conv"
+    r_name: str = "ra"
+    i_name: str = "ri"
+    lambda_name: str = "lam"
+    out_name: str = "o"
+    bias_suffix: str = ".b"
+
+
+@dataclasses.dataclass(frozen=True)
+class LayerScaleSpec:
+    """A weight per channel that a sublayer's (normed) result is multiplied by before it joins the stream."""
+
+    kind: str = "layer_scale"
+    size: int = 0
+    param_name: str = ""
+
+
+@dataclasses.dataclass(frozen=True)
 class ParallelMixerSpec:
-    """Two mixers side by side that read the same input; the result is left_scale * left + right_scale * right."""
+    """Two mixers side by side that read the same input; the result is left_scale * left + right_scale * right, or, with
+    ``out_norm_eps`` > 0, the same sum of the two results RMS-normed over the model width (weights left / right prefix +
+    ``out_norm_name``)."""
 
     kind: str = "parallel"
     left: Any = None
@@ -365,6 +411,8 @@ class ParallelMixerSpec:
     right_scale: float = 1.0
     left_name: str = "left."
     right_name: str = "right."
+    out_norm_eps: float = 0.0
+    out_norm_name: str = "out"
 
 
 @dataclasses.dataclass(frozen=True)
@@ -397,6 +445,11 @@ class BlockSpec:
     # ``post_norm`` are the norms of the two inputs, these the norms of the two results
     mixer_out_norm: Optional[NormSpec] = None
     feed_forward_out_norm: Optional[NormSpec] = None
+    # blocks that multiply a sublayer's normed result by a weight per channel (LayerScaleSpec)
+    mixer_scale: Any = None
+    feed_forward_scale: Any = None
+    mixer_scale_name: str = "ls1"
+    feed_forward_scale_name: str = "ls2"
     mixer_out_norm_name: str = "norm1b"
     feed_forward_out_norm_name: str = "norm2b"
 

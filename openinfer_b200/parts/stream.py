@@ -10,6 +10,8 @@ token's slice of a table all layers share, projected back, RMS-normed and added.
 "depth_average": after a layer, the stream becomes a weighted sum of the outputs of all layers so far and of the
 embedding output. It owns only the weights; the sum itself is formed by the kernel that ends the layer's last branch
 (``ops.branch_norm_add``) or by ``ops.history_average``.
+
+"layer_scale": a weight per channel on a sublayer's result.
 """
 from __future__ import annotations
 
@@ -22,7 +24,7 @@ from ..kernels import ops
 from .base import Part
 from .registry import register_stream_part
 from ..kernels.linear import linear
-from .spec import DepthAverageSpec, ParamInfo, ShortConvSpec, StreamCoefficientsSpec, TokenInputSpec
+from .spec import DepthAverageSpec, LayerScaleSpec, ParamInfo, ShortConvSpec, StreamCoefficientsSpec, TokenInputSpec
 
 
 @register_stream_part("short_conv")
@@ -65,6 +67,21 @@ class DepthAverage(Part):
     def parameters(self) -> Dict[str, ParamInfo]:
         s = self.spec
         return {s.param_name: ParamInfo((s.terms,), ("normal_around", 0.2, 1.0 / s.terms))}
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.weight = tensors[self.spec.param_name].contiguous()
+
+
+@register_stream_part("layer_scale")
+class LayerScale(Part):
+    """A weight per channel for a sublayer's normed result; the block multiplies it into the norm's weight."""
+
+    def __init__(self, spec: LayerScaleSpec) -> None:
+        super().__init__(spec)
+        self.weight: Optional[torch.Tensor] = None
+
+    def parameters(self) -> Dict[str, ParamInfo]:
+        return {self.spec.param_name: ParamInfo((self.spec.size,), ("normal_around", 0.1, 0.6))}
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         self.weight = tensors[self.spec.param_name].contiguous()
