@@ -160,16 +160,40 @@ def choose(z, correction, top: int, groups: int, keep: int):
     return s, torch.topk(c, top, dim=-1).indices
 
 
-def experts(h, p: Dict[str, torch.Tensor], pre: str, m: dict):
+def choice_margin(z, correction, top: int, groups: int, keep: int):
+    """[T]: how far every row's choice is from another one, in score units: the smaller of the gap between the last kept group
+    and the first one left out, and of the gap between the last chosen member and the best one left out."""
+    s, chosen = choose(z, correction, top, groups, keep)
+    c = s + correction
+    T, n = c.shape
+    best = c.view(T, groups, n // groups).max(dim=-1).values
+    margin = torch.full((T,), math.inf, dtype=c.dtype)
+    order = torch.sort(best, dim=-1, descending=True).values
+    if keep < groups:
+        margin = torch.minimum(margin, order[:, keep - 1] - order[:, keep])
+    kept = torch.zeros((T, groups), dtype=torch.bool)
+    kept.scatter_(1, torch.topk(best, keep, dim=-1).indices, True)
+    open_c = torch.where(kept.repeat_interleave(n // groups, dim=1), c, torch.full((), -math.inf, dtype=c.dtype))
+    ranked = torch.sort(open_c, dim=-1, descending=True).values
+    if top < (n // groups) * keep:
+        margin = torch.minimum(margin, ranked[:, top - 1] - ranked[:, top])
+    return margin
+
+
+def experts(h, p: Dict[str, torch.Tensor], pre: str, m: dict, margins: Optional[list] = None):
     r = m["router"]
     n, identity, top = int(r["experts"]), int(r.get("identity") or 0), int(r["top"])
     groups = r.get("groups") or {"count": 1, "keep": 1}
-    s, chosen = choose(h @ p[pre + "router"].T, p[pre + "correction"], top, int(groups["count"]), int(groups["keep"]))
+    z = h @ p[pre + "router"].T
+    s, chosen = choose(z, p[pre + "correction"], top, int(groups["count"]), int(groups["keep"]))
+    if margins is not None:
+        margins.append(choice_margin(z, p[pre + "correction"], top, int(groups["count"]), int(groups["keep"])))
+    scale = 1.0 if r.get("scale") is None else float(r["scale"])
     out = torch.zeros_like(h)
     for t in range(h.shape[0]):
         for e in chosen[t].tolist():
             y = h[t] if e >= n else gated_ff(h[t], p, f"{pre}e{e}.", silu)      # behind the experts: the input itself
-            out[t] += s[t, e] * float(r["scale"]) * y
+            out[t] += s[t, e] * scale * y
     if m.get("shared"):
         out = out + gated_ff(h, p, pre + "shared.", silu)
     assert n + identity == s.shape[1]
@@ -177,15 +201,16 @@ def experts(h, p: Dict[str, torch.Tensor], pre: str, m: dict):
 
 
 def forward(cfg: dict, p: Dict[str, torch.Tensor], tokens: List[int], layers_out: Optional[list] = None, dtype=torch.float64,
-            round_to=None, seen=None):
+            round_to=None, round_scale: float = 1.0, seen=None, margins: Optional[list] = None):
     """Logits [T, vocab] of one sequence in ``dtype``; ``layers_out`` collects the stream after every layer. ``round_to``:
     what the sublayers read, and an attention's queries, keys and values, are rounded to this type on the way (what a 16-bit
-    engine does at least). ``seen``: a mask in the place of every attention's own (a test asks what a lost key would do)."""
+    engine does at least), on a grid that ``round_scale`` stretches. ``seen``: a mask in the place of every attention's own (a test asks what a lost key would do);
+    ``margins`` collects how near every row's choice of experts was to another one."""
     p = {k: v.to(dtype) for k, v in p.items()}
     eps = float(cfg["norm"]["eps"])
 
     def read(x):
-        return x.to(round_to).to(dtype) if round_to is not None else x
+        return (x * round_scale).to(round_to).to(dtype) / round_scale if round_to is not None else x
 
     x = p["embed"][torch.tensor(tokens)] * float(cfg["embedding"]["scale"])
     for i, layer in enumerate(cfg["layers"]):
@@ -199,7 +224,7 @@ def forward(cfg: dict, p: Dict[str, torch.Tensor], tokens: List[int], layers_out
         x = x + layer_norm(a, p[pre + "norm1"], eps) * p[pre + "ls1"]      # norm and scale sit on the sublayer's output
         m = layer.get("mlp")
         if m:
-            f = gated_ff(read(x), p, pre + "mlp.", gelu_tanh) if m["kind"] == "dense" else experts(read(x), p, pre + "mlp.", m)
+            f = gated_ff(read(x), p, pre + "mlp.", gelu_tanh) if m["kind"] == "dense" else experts(read(x), p, pre + "mlp.", m, margins)
             x = x + layer_norm(f, p[pre + "norm2"], eps) * p[pre + "ls2"]
         if layers_out is not None:
             layers_out.append(x.clone())
