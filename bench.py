@@ -28,7 +28,9 @@ rotated key part under one norm with experts picked by a token table, a shared e
 fixed decay per head, attention normed behind its rotation under a window that keeps the first keys, latent attention whose
 cache a later layer reads, experts chosen by corrected sigmoid scores within the best groups),
 ``--design linurax`` for the Linurax design (norms on the sublayers' outputs, attention with sigmoid weights whose heads'
-scores are mixed and whose keys are its values, a gated recurrence per channel), beside Qwen3 and Delunex.
+scores are mixed and whose keys are its values, a gated recurrence per channel), beside Qwen3 and Delunex,
+``--design rolevik`` for the Rolevik design (attention in chunks beside a gated delta rule with a decay per head, a real-gated
+linear recurrent unit, experts of which some choices are the input itself), beside Qwen3, Pilonex and Linurax.
 """
 from __future__ import annotations
 
@@ -533,6 +535,31 @@ def linurax_configs(key, layers=None):
     return linurax, qwen, delunex
 
 
+def rolevik_configs(key, layers=None):
+    """Rolevik at the same widths and depths: every other layer is "parallel" (attention with per head 128 keys and values, a
+    quarter as many kv heads, half of each head rotated, in chunks of which a context of 2,048 is about in the middle; beside it a
+    gated delta rule of half as many heads behind four-tap filters), every other one a recurrent unit of one and a half times the
+    width in as many parts as there are heads; two layers with Qwen3's feed-forward take turns with two of sixteen experts of a
+    quarter of it and four choices that stand for the input, two of them a token in the two best of four groups, beside an expert
+    of that size that every token uses. Qwen3 as in ``design_configs``; beside it the engine's closest designs: Pilonex
+    (attention beside a delta rule, experts) and Linurax (norms on the sublayers' outputs, a recurrence per channel)."""
+    width, n_layers, heads, window, _, inter = DESIGN_SIZES[key]
+    n_layers = layers or n_layers
+    kv = max(1, heads // 4)
+    left = {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 21 * window // 16},
+            "rot": {"dims": 64, "base": 500000.0}}
+    right = {"heads": max(1, heads // 2), "kv_heads": kv, "dim": 128, "vdim": 128, "conv": 4}
+    experts = {"kind": "moe", "expert": {"ff": inter // 4}, "shared": {"ff": inter // 4},
+               "router": {"experts": 16, "identity": 4, "top": 2, "scale": 2.0, "groups": {"count": 4, "keep": 2}}}
+    lay = [{"type": "rglru", "mixer": {"width": 3 * width // 2, "blocks": heads, "conv": 4}} if i % 2 else
+           {"type": "parallel", "mixer": {"left": dict(left), "right": dict(right)}} for i in range(n_layers)]
+    for i, l in enumerate(lay):
+        l["mlp"] = dict(experts) if i % 4 > 1 else {"kind": "dense", "ff": inter}
+    rolevik = {"architecture": "Rolevik", "vocab": DESIGN_VOCAB, "width": width, "embedding": {"scale": 8.0}, "norm": {"eps": 1e-6},
+               "logit_scale": 0.5, "layers": lay}
+    return rolevik, design_configs(key, layers)[1], pilonex_configs(key, layers)[0], linurax_configs(key, layers)[0]
+
+
 def _part_tensors(torch, part, seen=None):
     """Every tensor a part holds, the tensors of parts inside it included."""
     seen = set() if seen is None else seen
@@ -549,9 +576,16 @@ def _part_tensors(torch, part, seen=None):
 
 
 def _attention_specs(mixer):
-    """(heads, cached row, window) of every paged attention inside a mixer."""
+    """(heads, cached row, what the cache was asked for) of every paged attention inside a mixer."""
     sides = [mixer.left, mixer.right] if hasattr(mixer, "left") else [mixer]
-    return [(m.spec.num_heads, m.kv_need().head_dim, m.kv_need().window) for m in sides if m.kv_need() is not None]
+    return [(m.spec.num_heads, m.kv_need().head_dim, m.kv_need()) for m in sides if m.kv_need() is not None]
+
+
+def _keys_seen(need, pos):
+    """Keys that the query at ``pos`` reads."""
+    if not need.window:
+        return pos + 1
+    return pos % need.window + 1 if need.chunked else min(pos + 1, need.window)
 
 
 class DesignBench:
@@ -646,14 +680,13 @@ class DesignBench:
                     if t is getattr(part, "table", None):          # a table indexed by the token id: one row a token
                         share = min(1.0, batch / t.shape[0])
                     if t.dim() == 3 and hasattr(part, "spec") and getattr(part.spec, "experts", 0):
-                        share = min(1.0, batch * part.spec.top / part.spec.experts)
+                        share = min(1.0, batch * part.spec.top / (part.spec.experts + part.spec.identity))
                     total += int(t.numel() * t.element_size() * share)
         total += model.head.numel() * model.head.element_size()
         for call, binding in zip(model.calls, model.bindings):
             need = model.blocks[call.layer].mixer.kv_need()
             if need is not None:
-                keys = min(self.context, need.window) if need.window else self.context
-                total += batch * keys * need.planes * need.num_kv_heads * need.head_dim * self.esize
+                total += batch * _keys_seen(need, self.context - 1) * need.planes * need.num_kv_heads * need.head_dim * self.esize
             for sid in binding.states:                  # recurrent state: one copy read, the other written
                 t = self.runner.cache.state_tensor(sid)
                 total += batch * t[0].numel() * t.element_size()
@@ -668,11 +701,12 @@ class DesignBench:
                 for v in _part_tensors(self.torch, part):
                     if v.dim() == 2 and v.shape[0] > 2 and v.shape[1] > 8:
                         flops += 2.0 * T * v.shape[0] * v.shape[1]
+                    elif v.dim() == 4:                                            # square matrices of a recurrent unit's parts
+                        flops += 2.0 * T * v.numel()
                     elif v.dim() == 3 and getattr(part.spec, "experts", 0):      # routed experts: `top` of them a row
-                        flops += 2.0 * T * part.spec.top * v.shape[1] * v.shape[2]
-            for heads, row, window in _attention_specs(block.mixer):
-                seen = sum(min(t + 1, window) if window else t + 1 for t in range(T))
-                flops += 4.0 * heads * row * seen
+                        flops += 2.0 * T * part.spec.top * part.spec.experts / (part.spec.experts + part.spec.identity) * v.shape[1] * v.shape[2]
+            for heads, row, need in _attention_specs(block.mixer):
+                flops += 4.0 * heads * row * sum(_keys_seen(need, t) for t in range(T))
             for m in (block.mixer, getattr(block.mixer, "left", None), getattr(block.mixer, "right", None)):
                 sp = getattr(m, "spec", None)
                 if sp is not None and getattr(sp, "kind", "") in ("matrix_memory", "gated_delta", "linear_attention"):   # memory update and read-out
@@ -712,9 +746,10 @@ def design_mode(args, torch, mods, peaks, peaks_src):
                 raise SystemExit(f"--design-sizes: unknown size {key!r} (known: {', '.join(DESIGN_SIZES)})")
             rec = {"width": DESIGN_SIZES[key][0], "layers": args.layers or DESIGN_SIZES[key][1]}
             configs = {"pilonex": pilonex_configs, "bubalix": bubalix_configs, "luzitar": luzitar_configs,
-                       "linurax": linurax_configs}.get(args.design, design_configs)(key, args.layers)
-            third = {"luzitar": "bubalix", "linurax": "delunex"}.get(args.design)      # the engine's closest design, where one is measured too
-            for arch, cfg in zip((args.design, "qwen3", third), configs):
+                       "linurax": linurax_configs, "rolevik": rolevik_configs}.get(args.design, design_configs)(key, args.layers)
+            # the engine's closest designs, where they are measured too
+            closest = {"luzitar": ("bubalix",), "linurax": ("delunex",), "rolevik": ("pilonex", "linurax")}.get(args.design, ())
+            for arch, cfg in zip((args.design, "qwen3", *closest), configs):
                 b = DesignBench(torch, mods, cfg, args.dtype, CONTEXT, 64, steps + warm + 16)
                 r = {"weights_gb": round(b.runner.model.weight_bytes() / 1e9, 3)}
                 for batch in (1, 8, 64):
@@ -774,7 +809,7 @@ def main() -> int:
     ap.add_argument("--profile", choices=["decode", "prefill", "mixed", "sampler"], default=None,
                     help="run warm-up, then ONE step between cudaProfilerStart/Stop and exit "
                          "(for `ncu --profile-from-start off`); prints no benchmark line")
-    ap.add_argument("--design", default=None, choices=["delunex", "pilonex", "bubalix", "luzitar", "linurax"],
+    ap.add_argument("--design", default=None, choices=["delunex", "pilonex", "bubalix", "luzitar", "linurax", "rolevik"],
                     help="instead of the headline workload: this design at layer sizes of real models beside Qwen3 at equal "
                          "sizes (decode at batch 1/8/64, a 2,048-token prefill), one JSON line")
     ap.add_argument("--design-sizes", default=None, help="sizes for --design, comma separated (1k, 2k, 4k; default 1k,2k)")
