@@ -9,7 +9,9 @@
 // u arrives as float32 sums. For 16-bit matrices it is split into two bfloat16 numbers, u = hi + lo (16 bits), and both halves
 // are multiplied with the same fragments of the matrices on the tensor cores (mma.sync m16n8k16, float32 accumulation): a block
 // takes 64 rows and 64 channels of one part, both matrices, 64 numbers of K at a time, the matrices by cp.async in two buffers.
-// float32 matrices take the ordinary pipes. Everything behind the products is float32 with the exact functions.
+// float32 matrices take the ordinary pipes. Everything behind the products is float32: with the exact functions for float32
+// results, with the special-function unit's exponential, division and root (a few units in the last place of float32) for
+// results that are rounded to 16 bits behind it.
 #include "oi_api.h"
 
 namespace {
@@ -43,12 +45,51 @@ __device__ __forceinline__ int single_slot(const GateArgs& p, int t) {
   return p.cu_seqlens[req + 1] - p.cu_seqlens[req] == 1 ? p.state_slots[req] : -1;
 }
 
+// exp(-|..|)-style coefficients of one number: a = exp(la) and sqrt(1 - a^2) for la <= 0
+template <bool kFast>
+__device__ __forceinline__ void decay_and_root(float la, float& a, float& root) {
+  if (!kFast) {
+    a = expf(la);
+    root = sqrtf(-expm1f(2.f * la));
+    return;
+  }
+  a = __expf(la);
+  // 1 - e^x, x = 2 la: near zero by its series (seven terms: below 2^-24 of it for |x| < 1/2), else as it stands
+  const float x = 2.f * la;
+  float p = 1.f + x * (1.f / 7.f);
+  p = 1.f + x * (1.f / 6.f) * p;
+  p = 1.f + x * (1.f / 5.f) * p;
+  p = 1.f + x * (1.f / 4.f) * p;
+  p = 1.f + x * (1.f / 3.f) * p;
+  p = 1.f + x * (1.f / 2.f) * p;
+  const float m = x > -0.5f ? -x * p : 1.f - a * a;
+  asm("sqrt.approx.ftz.f32 %0, %1;\n" : "=f"(root) : "f"(m));
+}
+template <bool kFast>
+__device__ __forceinline__ float sigmoid_f(float z) {
+  return kFast ? __fdividef(1.f, 1.f + __expf(-z)) : 1.f / (1.f + expf(-z));
+}
+
+// two neighbouring numbers of a row that leaves its coefficients for the scan
+__device__ __forceinline__ void finish_pair(const GateArgs& p, int t, int c, float zr0, float zi0, float zr1, float zi1) {
+  const int C = p.blocks * p.size;
+  const float2 br = *reinterpret_cast<const float2*>(p.bias + c), bi = *reinterpret_cast<const float2*>(p.bias + C + c);
+  const float2 rate = *reinterpret_cast<const float2*>(p.rate + c), u = *reinterpret_cast<const float2*>(p.u + (size_t)t * p.ld_u + c);
+  float2 a, root;
+  decay_and_root<true>(-sigmoid_f<true>(zr0 + br.x) * rate.x, a.x, root.x);
+  decay_and_root<true>(-sigmoid_f<true>(zr1 + br.y) * rate.y, a.y, root.y);
+  float* ab = p.ab + (size_t)t * p.ld_ab + c;
+  *reinterpret_cast<float2*>(ab) = a;
+  *reinterpret_cast<float2*>(ab + p.col_step) = make_float2(root.x * sigmoid_f<true>(zi0 + bi.x) * u.x, root.y * sigmoid_f<true>(zi1 + bi.y) * u.y);
+}
+
 template <typename TO>
 __device__ __forceinline__ void finish(const GateArgs& p, int t, int c, int slot, float zr, float zi) {
   const int C = p.blocks * p.size;
-  const float r = 1.f / (1.f + expf(-(zr + p.bias[c]))), i = 1.f / (1.f + expf(-(zi + p.bias[C + c])));
-  const float la = -r * p.rate[c];
-  const float a = expf(la), put = sqrtf(-expm1f(2.f * la)) * i * p.u[(size_t)t * p.ld_u + c];
+  constexpr bool kFast = sizeof(TO) == 2;
+  float a, root;
+  decay_and_root<kFast>(-sigmoid_f<kFast>(zr + p.bias[c]) * p.rate[c], a, root);
+  const float put = root * sigmoid_f<kFast>(zi + p.bias[C + c]) * p.u[(size_t)t * p.ld_u + c];
   if (slot == -1) {
     p.ab[(size_t)t * p.ld_ab + c] = a;
     p.ab[(size_t)t * p.ld_ab + p.col_step + c] = put;
@@ -103,6 +144,60 @@ __global__ void __launch_bounds__(256) rglru_gates_f32_kernel(const GateArgs p) 
   for (int i = 0; i < 4; ++i) {
     const int t = t0 + tm + 8 * i;
     if (t < p.tokens) finish<TO>(p, t, part * p.size + n0 + tn, single_slot(p, t), acc[0][i], acc[1][i]);
+  }
+}
+
+// bfloat16 matrices and few rows (single decoded tokens): a warp takes ONE channel, its rows of both matrices in registers (asked
+// for before the kernels ahead on the stream have finished), and walks the step's rows, 32 at a time, whose part of u lies in
+// shared memory; lane n ends row n.
+constexpr int kFewRows = 64, kFewSize = 512, kFewWarps = 8;
+
+__global__ void __launch_bounds__(kFewWarps * 32) rglru_gates_few_kernel(const GateArgs p) {
+  pdl_trigger();
+  extern __shared__ __align__(16) float us[];          // [32][size]
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int per = (p.size + kFewWarps - 1) / kFewWarps;
+  const int part = blockIdx.x / per, n = (blockIdx.x - part * per) * kFewWarps + warp;
+  const bool mine = n < p.size;
+  const bf16* w = reinterpret_cast<const bf16*>(p.w);
+  __nv_bfloat162 wr[kFewSize / 64], wi[kFewSize / 64];  // numbers 64 q + 2 lane, + 1 (p.vec: the size is a multiple of eight)
+  const __nv_bfloat162 zero = __floats2bfloat162_rn(0.f, 0.f);
+#pragma unroll
+  for (int q = 0; q < kFewSize / 64; ++q) {
+    const int k = 64 * q + 2 * lane;
+    const bool ok = mine && k < p.size;
+    const bf16* src = w + ((size_t)part * p.size + (ok ? n : 0)) * p.size + (ok ? k : 0);
+    wr[q] = ok ? *reinterpret_cast<const __nv_bfloat162*>(src) : zero;
+    wi[q] = ok ? *reinterpret_cast<const __nv_bfloat162*>(src + (size_t)p.blocks * p.size * p.size) : zero;
+  }
+  pdl_wait();
+  for (int t0 = 0; t0 < p.tokens; t0 += 32) {
+    const int rows = min(32, p.tokens - t0), quads = p.size / 4;
+    if (t0) __syncthreads();
+    for (int i = threadIdx.x; i < rows * quads; i += kFewWarps * 32) {
+      const int r = i / quads, c = (i - r * quads) * 4;
+      *reinterpret_cast<float4*>(us + r * p.size + c) = *reinterpret_cast<const float4*>(p.u + (size_t)(t0 + r) * p.ld_u + part * p.size + c);
+    }
+    const int slot = lane < rows ? single_slot(p, t0 + lane) : -3;
+    __syncthreads();
+    if (!mine) continue;
+    float zr = 0.f, zi = 0.f;
+    for (int r = 0; r < rows; ++r) {
+      float a = 0.f, b = 0.f;
+#pragma unroll
+      for (int q = 0; q < kFewSize / 64; ++q) {
+        const int k = 64 * q + 2 * lane;
+        if (64 * q < p.size) {
+          const float2 x = k < p.size ? *reinterpret_cast<const float2*>(us + r * p.size + k) : make_float2(0.f, 0.f);
+          const float2 fr = __bfloat1622float2(wr[q]), fi = __bfloat1622float2(wi[q]);
+          a += x.x * fr.x + x.y * fr.y;
+          b += x.x * fi.x + x.y * fi.y;
+        }
+      }
+      a = warp_sum(a), b = warp_sum(b);
+      if (lane == r) zr = a, zi = b;
+    }
+    if (lane < rows) finish<bf16>(p, t0 + lane, part * p.size + n, slot, zr, zi);
   }
 }
 
@@ -227,12 +322,17 @@ __global__ void __launch_bounds__(256) rglru_gates_mma_kernel(const GateArgs p) 
     if (t >= p.tokens) continue;
     const int slot = s.slot[m];
 #pragma unroll
-    for (int j = 0; j < 4; ++j)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int n = n0 + wn + 8 * j + 2 * tg + e;
-        if (n < p.size) finish<bf16>(p, t, part * p.size + n, slot, acc[0][j][2 * h + e], acc[1][j][2 * h + e]);
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + wn + 8 * j + 2 * tg;
+      if (p.vec && slot == -1) {         // (the size is a multiple of eight: both numbers or none)
+        if (n < p.size)
+          finish_pair(p, t, part * p.size + n, acc[0][j][2 * h], acc[1][j][2 * h], acc[0][j][2 * h + 1], acc[1][j][2 * h + 1]);
+        continue;
       }
+#pragma unroll
+      for (int e = 0; e < 2; ++e)
+        if (n + e < p.size) finish<bf16>(p, t, part * p.size + n + e, slot, acc[0][j][2 * h + e], acc[1][j][2 * h + e]);
+    }
   }
 }
 
@@ -263,7 +363,20 @@ OI_API int oi_rglru_gates(const float* u, long long ld_u, const void* w, int w_d
     OI_CHECK_LAUNCH();
     return OI_OK;
   }
-  p.vec = size % 8 == 0 && ld_u % 4 == 0 && ((uintptr_t)u & 15) == 0 && ((uintptr_t)w & 15) == 0;
+  p.vec = size % 8 == 0 && ld_u % 4 == 0 && ld_ab % 2 == 0 && col_step % 2 == 0 && ((uintptr_t)u & 15) == 0 && ((uintptr_t)w & 15) == 0 &&
+          ((uintptr_t)bias & 7) == 0 && ((uintptr_t)rate & 7) == 0 && ((uintptr_t)ab & 7) == 0;
+  // (batch-invariant mode: one kernel whatever the step's size)
+  if (p.vec && tokens <= kFewRows && size <= kFewSize && !oi_option(OI_OPT_BATCH_INVARIANT)) {
+    const size_t smem = (size_t)(tokens < 32 ? tokens : 32) * size * sizeof(float);
+    static bool few_configured = false;
+    if (!few_configured) {
+      OI_CHECK_CUDA(cudaFuncSetAttribute(rglru_gates_few_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 32 * kFewSize * (int)sizeof(float)));
+      few_configured = true;
+    }
+    oi_launch(rglru_gates_few_kernel, blocks * ((size + kFewWarps - 1) / kFewWarps), kFewWarps * 32, smem, s, p);
+    OI_CHECK_LAUNCH();
+    return OI_OK;
+  }
   const dim3 grid((tokens + kM - 1) / kM, blocks * ((size + kN - 1) / kN));
   static bool configured = false;
   if (!configured) {

@@ -444,9 +444,10 @@ __global__ void branch_join_kernel(const JoinArgs p) {
 // walks down its rows (rows of one request are consecutive), the taps' weights are read once, and only a request's
 // first rows of the step go to its state. The same launch leaves the new state: blocks behind the filter's own, one per
 // request, write the copy of the state that the step does not read.
-constexpr int kConvRows = 4;
+constexpr int kConvRows = 4;          // (steps of few rows, where a row's state is the longest wait: one row a thread)
+constexpr int kConvFewTokens = 128;
 constexpr int kConvMaxTaps = 8;
-template <typename TX, typename TO, int kTaps>     // kTaps: 2, 4 or 8, at least the taps
+template <typename TX, typename TO, int kTaps, int kRows>     // kTaps: 2, 4 or 8, at least the taps; kRows: rows a thread
 __global__ void __launch_bounds__(256) short_conv_vec_kernel(
     TO* __restrict__ out, const TX* __restrict__ x, const void* __restrict__ w, int w_dtype, float* __restrict__ state,
     long long state_stride, const int* __restrict__ cu_seqlens, const int* __restrict__ token_req,
@@ -483,7 +484,7 @@ __global__ void __launch_bounds__(256) short_conv_vec_kernel(
     }
     return;
   }
-  const int t0 = blockIdx.x * kConvRows;
+  const int t0 = blockIdx.x * kRows;
   float wt[kTaps][4];
   if (c < channels) {
 #pragma unroll
@@ -502,21 +503,21 @@ __global__ void __launch_bounds__(256) short_conv_vec_kernel(
     const int r = t0 - 1 - j;
     if (j < keep && r >= 0) load_in(x + (size_t)r * x_stride + c, ring[j]);
   }
-  const int t_end = min(tokens, t0 + kConvRows);
+  const int t_end = min(tokens, t0 + kRows);
   // The requests of the rows and of the taps - 1 rows above them, and the rows' inputs: all asked for before any is used.
   // A request's rows are consecutive, so a row's place in its portion shows in its neighbours' requests alone.
-  int reqs[kConvRows + kTaps - 1];
-  float curs[kConvRows][4];
+  int reqs[kRows + kTaps - 1];
+  float curs[kRows][4];
 #pragma unroll
-  for (int i = 0; i < kConvRows + kTaps - 1; ++i) {
+  for (int i = 0; i < kRows + kTaps - 1; ++i) {
     const int r = t0 - (kTaps - 1) + i;
     reqs[i] = (r >= 0 && r < t_end && r >= t0 - keep) ? token_req[r] : -2;
   }
 #pragma unroll
-  for (int i = 0; i < kConvRows; ++i)
+  for (int i = 0; i < kRows; ++i)
     if (t0 + i < t_end) load_in(x + (size_t)(t0 + i) * x_stride + c, curs[i]);
 #pragma unroll
-  for (int i = 0; i < kConvRows; ++i) {
+  for (int i = 0; i < kRows; ++i) {
     const int t = t0 + i;
     if (t >= t_end) break;
     const int req = reqs[i + kTaps - 1];
@@ -751,10 +752,11 @@ OI_API int oi_short_conv_strided(void* out, int out_dtype, long long out_stride,
                    (taps == 1 || (aligned16(state) && state_stride % 4 == 0)) && aligned16(in_bias) && aligned16(out_bias);
   const int vthreads = channels / 4 >= 256 ? 256 : ((channels / 4 + 31) / 32) * 32;
   // the filter's blocks, and behind them one block per request (and chunk of channels) that leaves the new state
-  const int conv_blocks = (tokens + kConvRows - 1) / kConvRows;
+  const bool few = tokens <= kConvFewTokens;
+  const int conv_rows = few ? 1 : kConvRows, conv_blocks = (tokens + conv_rows - 1) / conv_rows;
   const dim3 vgrid(conv_blocks + ((update_state && taps > 1) ? requests : 0), vec ? (channels / 4 + vthreads - 1) / vthreads : 1);
 #define OI_CONV_VEC(TX, TO, KT)                                                                                          \
-  oi_launch(short_conv_vec_kernel<TX, TO, KT>, vgrid, vthreads, 0, s, (TO*)out, (const TX*)x, w, w_dtype, state, state_stride, \
+  oi_launch(few ? short_conv_vec_kernel<TX, TO, KT, 1> : short_conv_vec_kernel<TX, TO, KT, kConvRows>, vgrid, vthreads, 0, s, (TO*)out, (const TX*)x, w, w_dtype, state, state_stride, \
             cu_seqlens, token_req, state_slots, state_phase, tokens, channels, taps, add_input, conv_blocks, x_stride, out_stride, act, \
             in_bias, out_bias)
 #define OI_CONV_CASE(XD, OD, TX, TO)                                                                                     \

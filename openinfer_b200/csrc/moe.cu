@@ -740,11 +740,12 @@ OI_API int oi_moe_route_scored(const void* x, int dtype, long long ldx, const vo
   if (rows == 0) return OI_OK;
   cudaStream_t s = (cudaStream_t)stream;
   const size_t smem = 3 * (size_t)all * sizeof(float) + (size_t)all + 16;
+  const int threads = all <= 16 ? 128 : (all >= 32 ? 256 : 32 * ((all + 3) / 4));      // a warp takes four experts at a time
   if (dtype == OI_F32)
-    oi_launch(moe_router_kernel<float>, rows, 128, smem, s, (const float*)x, ldx, w_router, w_dtype, rows, K, all, top, ids, wts, scoring,
+    oi_launch(moe_router_kernel<float>, rows, threads, smem, s, (const float*)x, ldx, w_router, w_dtype, rows, K, all, top, ids, wts, scoring,
               correction, n_groups, keep_groups, weight_scale);
   else if (dtype == OI_BF16)
-    oi_launch(moe_router_kernel<bf16>, rows, 128, smem, s, (const bf16*)x, ldx, w_router, w_dtype, rows, K, all, top, ids, wts, scoring,
+    oi_launch(moe_router_kernel<bf16>, rows, threads, smem, s, (const bf16*)x, ldx, w_router, w_dtype, rows, K, all, top, ids, wts, scoring,
               correction, n_groups, keep_groups, weight_scale);
   else
     OI_REQUIRE(false, "moe_route: unknown dtype code %d", dtype);

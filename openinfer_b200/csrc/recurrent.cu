@@ -117,14 +117,16 @@ __global__ void recurrent_prepare_kernel(ScanArgs a) {
 }
 
 // The records of the delta rule with one decay per head, by runs of four rows of a request (counted from its first row of the
-// step). With P_i the product of the decays from the run's first row to row i, R_im = g_i ... g_(i-m+1), and A the state in
-// front of the run,
-//   d_i = beta_i (v_i - P_i A^T k_i - sum_m R_im (k_(i-m) . k_i) d_(i-m)),
-//   o_i = P_i A^T q_i + (k_i . q_i) d_i + sum_m R_im (k_(i-m) . q_i) d_(i-m),      m = 1 .. i's place in its run,
+// step). With P_i the product of the decays from the run's first row to row i, R_ij = g_i ... g_(j+1), and A the state in front
+// of the run,
+//   d_i = beta_i (v_i - P_i A^T k_i - sum_(j < i) R_ij (k_j . k_i) d_j),
+//   o_i = P_i A^T q_i + sum_(j <= i) R_ij (k_j . q_i) d_j,        behind the run:  A <- P_3 A + sum_j R_3j k_j d_j,
 // so everything a run needs of the state are eight dot products with A that do not wait for one another; what is left between
-// its rows are numbers that no column of the state enters, and they are formed here. Record: keys [D] (unit), queries [D] (unit,
-// times q_scale), beta, P, R_1..3, R_m (k . k) 1..3, k . q, R_m (k . q) 1..3, padding.
+// its rows are numbers that no column of the state enters, and they are formed here. Record of row i: keys [D] (unit), queries
+// [D] (unit, times q_scale), then, on a 16-byte boundary, beta, P_i, g_i, R_ij (k_j . k_i) for j = 0..2, R_ij (k_j . q_i) for j = 0..3 (zero for j > i),
+// R_i(i-2), R_i(i-3), padding.
 constexpr int kDeltaScalars = 12;
+__host__ __device__ constexpr int delta_scalars_at(int D) { return (2 * D + 3) & ~3; }      // on a 16-byte boundary, whatever D is
 
 __global__ void delta_head_prepare_kernel(ScanArgs a) {
   pdl_start();
@@ -162,22 +164,30 @@ __global__ void delta_head_prepare_kernel(ScanArgs a) {
     const float rate = expf(load_as_f32(a.p1, a.p_dtype, h));
     decay = expf(-rate * softplus_f(a.gates[(size_t)(t - lane) * a.ld_gates + a.f_off + h] + load_as_f32(a.p0, a.p_dtype, h)));
   }
-  float R[4];
+  float R[4];                            // R[m]: the product over the row and the m rows above it
   R[0] = __shfl_sync(0xffffffffu, decay, 0);
 #pragma unroll
   for (int m = 1; m < 4; ++m) R[m] = R[m - 1] * __shfl_sync(0xffffffffu, decay, m);     // (one beyond the run's first row)
   if (lane == 0) {
-    float* s = rec + 2 * D;
+    float* s = rec + delta_scalars_at(D);
     s[0] = 1.f / (1.f + expf(-a.gates[(size_t)t * a.ld_gates + a.i_off + h]));
     s[1] = R[3];
-    s[8] = kq * kn * qn;
+    s[2] = R[0];
+    float ck[3] = {0.f, 0.f, 0.f}, cq[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-    for (int m = 0; m < 3; ++m) {
-      const float bn = m < place ? R[m] / sqrtf(n2[m] + 1e-6f) : 0.f;
-      s[2 + m] = R[m];
-      s[5 + m] = kk[m] * bn * kn;
-      s[9 + m] = kqs[m] * bn * qn;
+    for (int j = 0; j < 4; ++j) {
+      if (j == place) cq[j] = kq * kn * qn;
+#pragma unroll
+      for (int m = 0; m < 3; ++m)        // the row m + 1 above this one is the run's row place - 1 - m
+        if (place - 1 - m == j) {
+          const float bn = R[m] / sqrtf(n2[m] + 1e-6f);
+          cq[j] = kqs[m] * bn * qn;
+          if (j < 3) ck[j] = kk[m] * bn * kn;
+        }
     }
+    s[3] = ck[0], s[4] = ck[1], s[5] = ck[2];
+    s[6] = cq[0], s[7] = cq[1], s[8] = cq[2], s[9] = cq[3];
+    s[10] = R[1], s[11] = R[2];
   }
 }
 
@@ -436,28 +446,35 @@ __global__ void __launch_bounds__(kThreads) recurrent_scan_kernel(ScanArgs a, in
 }
 
 // The scan of the delta rule with one decay per head: blocks and staging as above, the request's rows four at a time (see
-// delta_head_prepare_kernel); what is left over one at a time.
+// delta_head_prepare_kernel), what is left over one at a time. kLanes lanes (16 or 32) hold TWO columns of the state, R numbers of
+// each a lane, so that a row's key and query are read once for both. The sixteen sums of a run over the lanes (two columns, four
+// rows, key or query) are formed by halving: every exchange leaves a lane half as many, until lane (column, row, kind) has its one.
 template <int kLanes, int R, bool kVec4>
 __global__ void __launch_bounds__(kThreads) delta_head_scan_kernel(ScanArgs a, int chunk) {
   pdl_wait();    // (no early trigger, as above)
   extern __shared__ __align__(16) float stage[];
-  constexpr int kCols = kThreads / kLanes;
+  constexpr int kCols = 2 * kThreads / kLanes;
   const int b = blockIdx.x, h = blockIdx.y;
   const int start = a.cu_seqlens[b], n_rows = a.cu_seqlens[b + 1] - start;
   if (n_rows <= 0 || a.token_req[start] < 0) return;
-  const int j = threadIdx.x % kLanes, cl = threadIdx.x / kLanes;
-  const int c = blockIdx.z * kCols + cl;
-  const bool col = c < a.V;
-  const int D = a.D, V = a.V, rec = a.rec;
+  const int lane = threadIdx.x & 31, j = threadIdx.x % kLanes, pair = threadIdx.x / kLanes;
+  const int c0 = blockIdx.z * kCols + 2 * pair;
+  const int D = a.D, V = a.V, rec = a.rec, at = delta_scalars_at(D);
   const int phase = a.state_phase[b];
   const float* old = a.state + (size_t)a.state_slots[b] * a.state_stride + ((size_t)phase * a.H + h) * D * V;
   float* fresh = a.state + (size_t)a.state_slots[b] * a.state_stride + ((size_t)(1 - phase) * a.H + h) * D * V;
-  float C[R];
+  float C[2][R];
 #pragma unroll
-  for (int i = 0; i < R; ++i) {
-    const int d = channel_of<kLanes, kVec4>(i, j);
-    C[i] = (col && d < D) ? old[(size_t)c * D + d] : 0.f;
-  }
+  for (int e = 0; e < 2; ++e)
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      const int d = channel_of<kLanes, kVec4>(i, j);
+      C[e][i] = (c0 + e < V && d < D) ? old[(size_t)(c0 + e) * D + d] : 0.f;
+    }
+  // which of a run's sums this lane ends up with, and where the sums with the keys of its column are
+  const int my_col = (j / (kLanes / 2)) & 1, my_row = (j / (kLanes / 8)) & 3;
+  const bool my_query = ((j / (kLanes / 16)) & 1) != 0, writer = my_query && (kLanes == 16 || (j & 1) == 0);
+  const int key_src = (lane & ~(kLanes - 1)) + my_col * (kLanes / 2);
   const int buf_floats = chunk * (rec + kCols);
   auto request = [&](int t0, int buf) {
     const int n = min(chunk, n_rows - t0), rec4 = rec / 4;
@@ -489,76 +506,106 @@ __global__ void __launch_bounds__(kThreads) delta_head_scan_kernel(ScanArgs a, i
     const float* vals = stage_now + (size_t)chunk * rec;
     int tt = 0;
     for (; tt + 3 < n; tt += 4) {
-      float k[4][R], ak[4], aq[4];
+      const float* run = stage_now + (size_t)tt * rec;
+      float k[4][R], v[16];
 #pragma unroll
       for (int u = 0; u < 4; ++u) {
-        const float* r = stage_now + (size_t)(tt + u) * rec;
         float q[R];
-        load_channels<kLanes, R, kVec4>(k[u], r, D, j);
-        load_channels<kLanes, R, kVec4>(q, r + D, D, j);
-        float pk[2] = {0.f, 0.f}, pq[2] = {0.f, 0.f};
+        load_channels<kLanes, R, kVec4>(k[u], run + (size_t)u * rec, D, j);
+        load_channels<kLanes, R, kVec4>(q, run + (size_t)u * rec + D, D, j);
 #pragma unroll
-        for (int i = 0; i < R; ++i) {
-          pk[i & 1] += C[i] * k[u][i];
-          pq[i & 1] += C[i] * q[i];
+        for (int e = 0; e < 2; ++e) {
+          float pk[2] = {0.f, 0.f}, pq[2] = {0.f, 0.f};
+#pragma unroll
+          for (int i = 0; i < R; ++i) {
+            pk[i & 1] += C[e][i] * k[u][i];
+            pq[i & 1] += C[e][i] * q[i];
+          }
+          v[(e * 4 + u) * 2] = pk[0] + pk[1];
+          v[(e * 4 + u) * 2 + 1] = pq[0] + pq[1];
         }
-        ak[u] = pk[0] + pk[1], aq[u] = pq[0] + pq[1];
       }
-#pragma unroll
-      for (int u = 0; u < 4; ++u) ak[u] = lanes_sum<kLanes>(ak[u]), aq[u] = lanes_sum<kLanes>(aq[u]);
-      float d[4], o[4];
+      // the run's numbers that wait for no sum
+      float4 s0[4], s1[4];
 #pragma unroll
       for (int u = 0; u < 4; ++u) {
-        const float* s = stage_now + (size_t)(tt + u) * rec + 2 * D;
-        float want = vals[(tt + u) * kCols + cl] - s[1] * ak[u];
-        o[u] = s[1] * aq[u];
-#pragma unroll
-        for (int m = 0; m < u; ++m) {
-          want -= s[5 + m] * d[u - 1 - m];
-          o[u] += s[9 + m] * d[u - 1 - m];
-        }
-        d[u] = s[0] * want;
-        o[u] += s[8] * d[u];
+        s0[u] = *reinterpret_cast<const float4*>(run + (size_t)u * rec + at);       // beta, P, g, ck0
+        s1[u] = *reinterpret_cast<const float4*>(run + (size_t)u * rec + at + 4);   // ck1, ck2, cq0, cq1
       }
-      const float* last = stage_now + (size_t)(tt + 3) * rec + 2 * D;
-      const float keep = last[1], w0 = d[0] * last[4], w1 = d[1] * last[3], w2 = d[2] * last[2];
+      const float* own = run + (size_t)my_row * rec + at;
+      const float own_P = own[1], cq0 = own[6], cq1 = own[7], cq2 = own[8], cq3 = own[9];
+      const float4 tail = *reinterpret_cast<const float4*>(run + (size_t)3 * rec + at + 8);   // cq2, cq3, R_31, R_30
+      float want[4];
 #pragma unroll
-      for (int i = 0; i < R; ++i) C[i] = keep * C[i] + ((k[0][i] * w0 + k[1][i] * w1) + (k[2][i] * w2 + k[3][i] * d[3]));
-      if (j == 0 && col) {
-        float* o_row = a.out + (size_t)(start + t0 + tt) * a.ld_out + (size_t)h * V + c;
+      for (int u = 0; u < 4; ++u) want[u] = vals[(tt + u) * kCols + 2 * pair + my_col];
+      // halving: column, row, row, kind
 #pragma unroll
-        for (int u = 0; u < 4; ++u) o_row[(size_t)u * a.ld_out] = o[u];
+      for (int half = 8, o = kLanes / 2; half > 0; half >>= 1, o >>= 1) {
+        const bool up = (j & o) != 0;
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+          if (i < half) {
+            const float send = up ? v[i] : v[i + half], keep = up ? v[i + half] : v[i];
+            v[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+          }
+      }
+      if (kLanes == 32) v[0] += __shfl_xor_sync(0xffffffffu, v[0], 1);
+      float ak[4], d[4], dx[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) ak[u] = __shfl_sync(0xffffffffu, v[0], key_src + u * (kLanes / 8));
+      d[0] = s0[0].x * (want[0] - s0[0].y * ak[0]);
+      d[1] = s0[1].x * (want[1] - s0[1].y * ak[1] - s0[1].w * d[0]);
+      d[2] = s0[2].x * (want[2] - s0[2].y * ak[2] - s0[2].w * d[0] - s1[2].x * d[1]);
+      d[3] = s0[3].x * (want[3] - s0[3].y * ak[3] - s0[3].w * d[0] - s1[3].x * d[1] - s1[3].y * d[2]);
+      if (writer && c0 + my_col < V)
+        a.out[(size_t)(start + t0 + tt + my_row) * a.ld_out + (size_t)h * V + c0 + my_col] =
+            own_P * v[0] + (cq0 * d[0] + cq1 * d[1]) + (cq2 * d[2] + cq3 * d[3]);
+      d[0] *= tail.w, d[1] *= tail.z, d[2] *= s0[3].z;
+#pragma unroll
+      for (int u = 0; u < 4; ++u) dx[u] = __shfl_xor_sync(0xffffffffu, d[u], kLanes / 2);    // the other column's
+      const float keep = s0[3].y;
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const bool mine = my_col == e;
+        const float w0 = mine ? d[0] : dx[0], w1 = mine ? d[1] : dx[1], w2 = mine ? d[2] : dx[2], w3 = mine ? d[3] : dx[3];
+#pragma unroll
+        for (int i = 0; i < R; ++i) C[e][i] = keep * C[e][i] + ((k[0][i] * w0 + k[1][i] * w1) + (k[2][i] * w2 + k[3][i] * w3));
       }
     }
     for (; tt < n; ++tt) {
       const float* r = stage_now + (size_t)tt * rec;
-      const float beta = r[2 * D], g = r[2 * D + 2];
+      const float beta = r[at], g = r[at + 2];
       float k[R], q[R];
       load_channels<kLanes, R, kVec4>(k, r, D, j);
       load_channels<kLanes, R, kVec4>(q, r + D, D, j);
-      float kv[2] = {0.f, 0.f};
 #pragma unroll
-      for (int i = 0; i < R; ++i) {
-        C[i] *= g;
-        kv[i & 1] += C[i] * k[i];
-      }
-      const float dlt = beta * (vals[tt * kCols + cl] - lanes_sum<kLanes>(kv[0] + kv[1]));
-      float num[2] = {0.f, 0.f};
+      for (int e = 0; e < 2; ++e) {
+        float kv[2] = {0.f, 0.f};
 #pragma unroll
-      for (int i = 0; i < R; ++i) {
-        C[i] += k[i] * dlt;
-        num[i & 1] += C[i] * q[i];
+        for (int i = 0; i < R; ++i) {
+          C[e][i] *= g;
+          kv[i & 1] += C[e][i] * k[i];
+        }
+        const float dlt = beta * (vals[tt * kCols + 2 * pair + e] - lanes_sum<kLanes>(kv[0] + kv[1]));
+        float num[2] = {0.f, 0.f};
+#pragma unroll
+        for (int i = 0; i < R; ++i) {
+          C[e][i] += k[i] * dlt;
+          num[i & 1] += C[e][i] * q[i];
+        }
+        const float o = lanes_sum<kLanes>(num[0] + num[1]);
+        if (j == 0 && c0 + e < V) a.out[(size_t)(start + t0 + tt) * a.ld_out + (size_t)h * V + c0 + e] = o;
       }
-      const float o = lanes_sum<kLanes>(num[0] + num[1]);
-      if (j == 0 && col) a.out[(size_t)(start + t0 + tt) * a.ld_out + (size_t)h * V + c] = o;
     }
     __syncthreads();                           // everyone has read this buffer before the chunk after next is requested into it
   }
 #pragma unroll
-  for (int i = 0; i < R; ++i) {
-    const int d = channel_of<kLanes, kVec4>(i, j);
-    if (col && d < D) fresh[(size_t)c * D + d] = C[i];
-  }
+  for (int e = 0; e < 2; ++e)
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+      const int d = channel_of<kLanes, kVec4>(i, j);
+      if (c0 + e < V && d < D) fresh[(size_t)(c0 + e) * D + d] = C[e][i];
+    }
 }
 
 // out[t, h, c] = o[t, h, c] * rsqrt(mean_c o[t, h, :]^2 + eps) * w[h * w_stride + c] * act(gate[t, h, c]) * scale, act the
@@ -607,7 +654,7 @@ __global__ void row_norm_gate_kernel(TO* __restrict__ out, long long ld_out, con
 
 // floats of scratch the scan wants per row: oi_recurrent_scan's `prep` is [tokens, H, that]
 OI_API int oi_recurrent_record(int mode, int D) {                        // a multiple of four floats: 16-byte copies
-  return mode == kDeltaHeadDecay ? (2 * D + kDeltaScalars + 3) & ~3 : (3 * D + 2 + 3) & ~3;
+  return mode == kDeltaHeadDecay ? delta_scalars_at(D) + kDeltaScalars : (3 * D + 2 + 3) & ~3;
 }
 
 // mode 0: matrix memory (p0, p1: the two gate biases [H]); mode 1: gated delta rule (p0: dt [H * D], p1: A [H];
@@ -647,18 +694,16 @@ OI_API int oi_recurrent_scan(int mode, const float* qkv, long long ld_qkv, int q
     const int rows = D <= 128 ? 16 : (D <= 256 ? 8 : 4);       // per buffer: two buffers of at most 19 KB
 #define OI_DELTA_HEAD(LANES, REGS)                                                                                          \
   do {                                                                                                                      \
-    constexpr int cols = kThreads / LANES;                                                                                  \
+    constexpr int cols = 2 * kThreads / LANES;                                                                              \
     const dim3 grid(requests, H, (V + cols - 1) / cols);                                                                    \
     const size_t smem = 2 * (size_t)rows * (a.rec + cols) * sizeof(float);                                                  \
     oi_fence_next_launch();      /* plain stream order, as below */                                                         \
     if (D % 4 == 0) oi_launch(delta_head_scan_kernel<LANES, REGS, true>, grid, kThreads, smem, s, a, rows);                 \
     else oi_launch(delta_head_scan_kernel<LANES, REGS, false>, grid, kThreads, smem, s, a, rows);                           \
   } while (0)
-    if (D <= 16) OI_DELTA_HEAD(4, 4);
-    else if (D <= 32) OI_DELTA_HEAD(8, 4);
-    else if (D <= 64) OI_DELTA_HEAD(8, 8);
-    else if (D <= 128) OI_DELTA_HEAD(8, 16);
-    else if (D <= 256) OI_DELTA_HEAD(16, 16);
+    if (D <= 64) OI_DELTA_HEAD(16, 4);
+    else if (D <= 128) OI_DELTA_HEAD(32, 4);
+    else if (D <= 256) OI_DELTA_HEAD(32, 8);
     else OI_DELTA_HEAD(32, 16);
 #undef OI_DELTA_HEAD
     OI_CHECK_LAUNCH();
