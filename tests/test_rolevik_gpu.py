@@ -179,7 +179,7 @@ def test_attention_kernels_under_chunks(nq, nkv, hd, chunk):
                 assert err < (2e-5 if td == torch.float32 else 3e-2), f"{td} tcgen05 {tcgen} page {page} request {b}: {err}"
 
 
-@pytest.mark.parametrize("H,G,D,V", [(4, 2, 16, 24), (3, 1, 7, 5), (2, 2, 64, 40), (1, 1, 20, 3), (4, 1, 128, 64), (2, 1, 200, 8), (1, 1, 300, 16), (5, 5, 32, 17)])
+@pytest.mark.parametrize("H,G,D,V", [(4, 2, 16, 24), (3, 1, 7, 5), (2, 2, 64, 40), (1, 1, 20, 3), (4, 1, 128, 64), (2, 1, 200, 8), (1, 1, 300, 16), (5, 5, 32, 17), (20, 5, 96, 128), (24, 24, 48, 130)])
 def test_delta_rule_with_a_decay_per_head_kernel(H, G, D, V):
     """Portions over old state beside single tokens and a padding request: runs of four rows, what is left over, both copies of
     the state; strong and weak decays, queries and keys of any length."""
@@ -665,16 +665,17 @@ def test_greedy_generation_through_the_scheduler(folders, name):
     assert llm16.runner.cache.slot_pool.used_count == 0
 
 
-def test_batch_invariant_mode_is_bitwise(folders):
+@pytest.mark.parametrize("name", ["C", "E", "F"])
+def test_batch_invariant_mode_is_bitwise(folders, name):
     """In batch-invariant mode a request's bfloat16 logits are the same bit for bit alone and among others."""
     from openinfer_b200.engine.runner import StepEntry
     from openinfer_b200.kernels import policy
-    cfg = CASES["F"][0]
+    cfg = CASES[name][0]
     reqs = {f"b{i}": tokens_for(cfg, n, 90 + i) for i, n in enumerate([40, 65, 1, 33])}
     policy.set_batch_invariant(True)
     try:
         def run(ids):
-            runner = runner_for(folders["F", "bfloat16"], "bfloat16", max_tokens=512)
+            runner = runner_for(folders[name, "bfloat16"], "bfloat16", max_tokens=512)
             rows = {r: [] for r in ids}
             for part in (slice(0, 20), slice(20, 33)):
                 entries = [StepEntry(r, reqs[r][part], list(range(len(reqs[r][part])))) for r in ids if reqs[r][part]]
