@@ -21,7 +21,7 @@
 // recorded and replayed. A row's sums are formed in the same order whatever else shares its tile: the result of a row does
 // not depend on the batch. The tiles' products run on the tensor cores for bfloat16 operands (mma.sync, float32
 // accumulation) and on the ordinary pipes for float32 and for rows that cannot be read 16 bytes at a time.
-#include "common.cuh"
+#include "oi_api.h"
 
 namespace {
 
@@ -710,7 +710,8 @@ OI_API int oi_moe_max_tiles(int pairs, int experts) { return pairs / kTileM + ex
 OI_API int oi_moe_tile_rows(int pairs, int experts) { return (long long)pairs >= 64LL * experts ? kBigM : kTileM; }
 
 // Steps of at most this many (row, choice) pairs take the row-by-row products and need no grouping.
-OI_API int oi_moe_small(int pairs, int experts) { return pairs <= 2 * experts && pairs <= 64; }
+// (None in batch-invariant mode, where a row's sums must be formed the same way whatever else is in the step.)
+OI_API int oi_moe_small(int pairs, int experts) { return !oi_option(OI_OPT_BATCH_INVARIANT) && pairs <= 2 * experts && pairs <= 64; }
 
 // x [rows, K] (row stride ldx) in `dtype`; router weights [E, K]; ids, wts [rows, top]; sorted [rows * top];
 // tile_info [3 * max_tiles + 1] with max_tiles = oi_moe_max_tiles(rows * top, E).

@@ -665,7 +665,7 @@ def test_greedy_generation_through_the_scheduler(folders, name):
     assert llm16.runner.cache.slot_pool.used_count == 0
 
 
-@pytest.mark.parametrize("name", ["C", "E", "F"])
+@pytest.mark.parametrize("name", ["C", "F"])
 def test_batch_invariant_mode_is_bitwise(folders, name):
     """In batch-invariant mode a request's bfloat16 logits are the same bit for bit alone and among others."""
     from openinfer_b200.engine.runner import StepEntry
